@@ -464,6 +464,14 @@ int32_t kanso_cuda_model_load(kanso_cuda_ctx* ctx, const char* dir, int32_t comp
  * kanso_cuda_kv_create's, its layers may differ in heads and in key and value size. */
 int32_t kanso_cuda_model_create_pool(kanso_cuda_model* m, uint32_t num_blocks,
                                      kanso_cuda_kv** out);
+/* The same with a number of state slots. A model with recurrent layers keeps, besides the pages,
+ * one state per live sequence and layer; the host gives each live sequence a slot of its own.
+ * (Without this call: as many as pages, at most 256.) A slot needs no clearing between sequences:
+ * a sequence's first token reads no state. */
+int32_t kanso_cuda_model_create_pool_slots(kanso_cuda_model* m, uint32_t num_blocks,
+                                           uint32_t num_slots, kanso_cuda_kv** out);
+/* Bytes of one slot, all layers. */
+uint64_t kanso_cuda_kv_state_bytes(const kanso_cuda_kv* kv);
 /* A ragged step, any model class: sequence s brings query_lens[s] tokens, the last ones of its
  * context_lens[s]; earlier ones lie in the pool. tokens u32[sum query_lens]; block_tables
  * u32[S*max_blocks]; want u32[n_want] = rows of the step (0 .. sum query_lens - 1); all HOST.
@@ -474,6 +482,22 @@ int32_t kanso_cuda_forward_step(kanso_cuda_ctx* ctx, kanso_cuda_model* m, kanso_
                                 const uint32_t* context_lens, const uint32_t* block_tables,
                                 uint32_t S, uint32_t max_blocks, const uint32_t* want,
                                 uint32_t n_want, float* logits_out);
+/* The two steps for models with recurrent layers: sequence s has its state in slot state_slots[s]
+ * (HOST u32[S] in the first, device u32[B] in the second; no slot twice). NULL, and the calls
+ * without the argument: sequence s has slot s. */
+int32_t kanso_cuda_forward_step_slots(kanso_cuda_ctx* ctx, kanso_cuda_model* m, kanso_cuda_kv* kv,
+                                      const uint32_t* tokens, const uint32_t* query_lens,
+                                      const uint32_t* context_lens, const uint32_t* block_tables,
+                                      const uint32_t* state_slots, uint32_t S, uint32_t max_blocks,
+                                      const uint32_t* want, uint32_t n_want, float* logits_out);
+int32_t kanso_cuda_decode_step_device_slots(kanso_cuda_ctx* ctx, kanso_cuda_model* m,
+                                            kanso_cuda_kv* kv, const uint32_t* tokens,
+                                            const uint32_t* positions, const uint32_t* slots,
+                                            const uint32_t* block_tables,
+                                            const uint32_t* context_lens,
+                                            const uint32_t* state_slots, uint32_t B,
+                                            uint32_t max_blocks, uint32_t max_ctx,
+                                            int32_t act_mode, float* logits_dev);
 
 /* ------------------------------------------------------------------------- */
 /* Engine: the cache pages of live requests, ragged batches over them, and greedy generation. */
@@ -530,6 +554,16 @@ int32_t kanso_cuda_kv_create_dense(kanso_cuda_ctx* ctx, uint32_t num_layers,
                                    const uint32_t* kv_heads, const uint32_t* k_dim,
                                    const uint32_t* v_dim, uint32_t num_blocks,
                                    uint32_t block_size, int32_t kv_type, kanso_cuda_kv** out);
+/* The same layer by layer: rows per token (kv_heads 0: none; v_dim 0: key rows only, as latent
+ * attention keeps them) and a recurrent state per slot (state_heads 0: none). */
+typedef struct kanso_kv_layer {
+  uint32_t kv_heads, k_dim, v_dim;
+  uint32_t state_heads, state_dim, state_vdim;
+} kanso_kv_layer;
+int32_t kanso_cuda_kv_create_layers(kanso_cuda_ctx* ctx, uint32_t num_layers,
+                                    const kanso_kv_layer* layers, uint32_t num_blocks,
+                                    uint32_t block_size, int32_t kv_type, uint32_t num_slots,
+                                    kanso_cuda_kv** out);
 /* RMS norm over the whole q row and the whole k row of qkv f32[T][H*k_dim + G*k_dim + G*v_dim],
  * then k and v to their places in the pool and q to q_out [T][num_heads][k_dim rounded up to 8]. */
 int32_t kanso_cuda_qk_norm_store(kanso_cuda_ctx* ctx, kanso_cuda_kv* kv, uint32_t layer,

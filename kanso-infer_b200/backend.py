@@ -132,6 +132,13 @@ PROTOTYPES = {
     "kanso_cuda_model_describe": (_I32, [C.c_char_p, C.c_char_p, _SZ]),
     "kanso_cuda_model_load": (_I32, [_P, C.c_char_p, _I32, C.POINTER(_P)]),
     "kanso_cuda_model_create_pool": (_I32, [_P, _U32, C.POINTER(_P)]),
+    "kanso_cuda_model_create_pool_slots": (_I32, [_P, _U32, _U32, C.POINTER(_P)]),
+    "kanso_cuda_kv_state_bytes": (_U64, [_P]),
+    "kanso_cuda_kv_create_layers": (_I32, [_P, _U32, _P, _U32, _U32, _I32, _U32, C.POINTER(_P)]),
+    "kanso_cuda_forward_step_slots": (_I32, [_P, _P, _P, _P, _P, _P, _P, _P, _U32, _U32, _P, _U32,
+                                             _P]),
+    "kanso_cuda_decode_step_device_slots": (_I32, [_P, _P, _P, _P, _P, _P, _P, _P, _P, _U32, _U32,
+                                                   _U32, _I32, _P]),
     "kanso_cuda_forward_step": (_I32, [_P, _P, _P, _P, _P, _P, _P, _U32, _U32, _P, _U32, _P]),
     "kanso_cuda_engine_create": (_I32, [_P, _U32, _U32, C.POINTER(_P)]),
     "kanso_cuda_engine_destroy": (_I32, [_P]),
@@ -325,12 +332,14 @@ class KvPool:
         self.h = h
 
     @classmethod
-    def of_model(cls, model: "Model", num_blocks: int):
+    def of_model(cls, model: "Model", num_blocks: int, num_slots: int | None = None):
         self = cls.__new__(cls)
         self.ctx, self.geom = model.ctx, None
         h = _P()
-        model.ctx.check(model.ctx.lib.kanso_cuda_model_create_pool(model.h, num_blocks,
-                                                                   C.byref(h)))
+        lib = model.ctx.lib
+        model.ctx.check(
+            lib.kanso_cuda_model_create_pool(model.h, num_blocks, C.byref(h)) if num_slots is None
+            else lib.kanso_cuda_model_create_pool_slots(model.h, num_blocks, num_slots, C.byref(h)))
         self.h = h
         return self
 
@@ -342,6 +351,18 @@ class KvPool:
         h = _P()
         ctx.call("kanso_cuda_kv_create_dense", len(kv_heads), _ptr(kv_heads), _ptr(k_dim),
                  _ptr(v_dim), num_blocks, block_size, kv_type, C.byref(h))
+        self.h = h
+        return self
+
+    @classmethod
+    def of_layers(cls, ctx: Context, layers, num_blocks, block_size, kv_type, num_slots=0):
+        """An unquantised pool; layers is a uint32 array [n, 6] of kv_heads, k_dim, v_dim (0: no
+        rows) and state_heads, state_dim, state_vdim (0: no state)."""
+        self = cls.__new__(cls)
+        self.ctx, self.geom = ctx, None
+        h = _P()
+        ctx.call("kanso_cuda_kv_create_layers", len(layers), _ptr(layers), num_blocks, block_size,
+                 kv_type, num_slots, C.byref(h))
         self.h = h
         return self
 
@@ -377,6 +398,11 @@ class KvPool:
     @property
     def bytes_per_token(self) -> int:
         return self.ctx.lib.kanso_cuda_kv_bytes_per_token(self.h)
+
+    @property
+    def state_bytes(self) -> int:
+        """Bytes of one sequence's recurrent state, all layers."""
+        return self.ctx.lib.kanso_cuda_kv_state_bytes(self.h)
 
     def paged_attention(self, layer, q, block_tables, context_lens, out,
                         params: PagedAttentionParams, host_context_lens=None):
@@ -437,9 +463,9 @@ class Model:
         self.h = h
         return self
 
-    def create_pool(self, num_blocks: int) -> "KvPool":
+    def create_pool(self, num_blocks: int, num_slots: int | None = None) -> "KvPool":
         """A pool of the geometry and element type the model's step reads."""
-        return KvPool.of_model(self, num_blocks)
+        return KvPool.of_model(self, num_blocks, num_slots)
 
     def destroy(self):
         if getattr(self, "h", None):
@@ -468,17 +494,18 @@ class Model:
                       max_blocks, act_mode, _ptr(logits_out))
 
     def decode_step_device(self, kv: KvPool, tokens, positions, slots, block_tables,
-                           context_lens, B, max_blocks, max_ctx, logits, act_mode=ACT_F32):
-        self.ctx.call("kanso_cuda_decode_step_device", self.h, kv.h, _ptr(tokens),
-                      _ptr(positions), _ptr(slots), _ptr(block_tables), _ptr(context_lens), B,
-                      max_blocks, max_ctx, act_mode, _ptr(logits))
+                           context_lens, B, max_blocks, max_ctx, logits, act_mode=ACT_F32,
+                           state_slots=None):
+        self.ctx.call("kanso_cuda_decode_step_device_slots", self.h, kv.h, _ptr(tokens),
+                      _ptr(positions), _ptr(slots), _ptr(block_tables), _ptr(context_lens),
+                      _ptr(state_slots), B, max_blocks, max_ctx, act_mode, _ptr(logits))
 
     def forward_step(self, kv: KvPool, tokens, query_lens, context_lens, block_tables, max_blocks,
-                     want, logits_out):
+                     want, logits_out, state_slots=None):
         """A ragged step; HOST numpy arrays (uint32 / float32); synchronous."""
-        self.ctx.call("kanso_cuda_forward_step", self.h, kv.h, _ptr(tokens), _ptr(query_lens),
-                      _ptr(context_lens), _ptr(block_tables), len(query_lens), max_blocks,
-                      _ptr(want), len(want), _ptr(logits_out))
+        self.ctx.call("kanso_cuda_forward_step_slots", self.h, kv.h, _ptr(tokens),
+                      _ptr(query_lens), _ptr(context_lens), _ptr(block_tables), _ptr(state_slots),
+                      len(query_lens), max_blocks, _ptr(want), len(want), _ptr(logits_out))
 
 
 def describe_model(path: str) -> dict:

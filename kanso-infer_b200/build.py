@@ -27,9 +27,10 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
 
 # What a library that serves one model class is made of; the full library has every source.
 CORE = ["ctx", "kv_pool", "glue", "model_api", "safetensors", "engine"]
+DENSE = ["dense_model", "dense_rows", "gemv_dense", "gemm_dense"]  # the unquantised classes
 MODEL_CLASSES = {
-    "Revitar": ["revitar", "dense_rows", "gemv_dense", "gemm_dense", "sigmoid_attention",
-                "sigmoid_prefill"],
+    "Revitar": ["revitar", *DENSE, "sigmoid_attention", "sigmoid_prefill"],
+    "Migurax": ["migurax", *DENSE, "latent_attention", "softmax_prefill", "mlstm"],
 }
 
 

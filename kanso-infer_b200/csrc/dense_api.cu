@@ -204,7 +204,8 @@ int32_t kanso_cuda_moe(kanso_cuda_ctx* ctx, int32_t compute, const float* x, con
     GemvSource src;
     src.x = x;
     st = launch_gemv(ctx, KANSO_COMPUTE_F32, r, src, rl, experts, (int)T);
-    if (!st) st = launch_gemv_gate_up(ctx, compute, g, u, x, rl, experts, top, a32, sel, (int)T);
+    if (!st) st = launch_gemv_gate_up(ctx, compute, &g, u, x, rl, experts, top, RouteWeights::kShares,
+                                        a32, sel, (int)T);
     if (!st) st = launch_gemv_down(ctx, compute, d, a32, sel, top, y, (int)T);
   } else {
     if (compute == KANSO_COMPUTE_BF16)
@@ -212,7 +213,8 @@ int32_t kanso_cuda_moe(kanso_cuda_ctx* ctx, int32_t compute, const float* x, con
     else
       narrow_kernel<float><<<256, 256, 0, ctx->stream>>>(x, (float*)(mem + o_xe), T, WL, width);
     st = after_launch(ctx, "narrow");
-    if (!st) st = launch_route(ctx, x, width, r, top, sel, wgt, cnt, slot, T);
+    if (!st) st = launch_route(ctx, x, width, r, nullptr, top, RouteWeights::kShares, sel, wgt,
+                              cnt, slot, T);
     if (!st)
       st = launch_expert_gather(ctx, compute, cnt, experts, top, sel, slot, off, mem + o_xe, WL,
                                 mem + o_xs, T);

@@ -2,6 +2,8 @@
 // x += mult * rmsnorm(y) * w, the norm of wanted rows, q / k norm with the store to the pool, and
 // the routing of rows to experts. All of it in 32-bit; what feeds a matrix product is also
 // written in the product's element type.
+#include <cmath>
+
 #include "dense.cuh"
 
 namespace kanso {
@@ -46,14 +48,15 @@ __device__ __forceinline__ void store4(float* p, float a, float b, float c, floa
 template <typename E>
 __global__ void __launch_bounds__(DR_THREADS)
     residual_norm_kernel(float* __restrict__ x, int width, const ResidualSource s,
-                         const float* __restrict__ w, float eps, float mult, E* __restrict__ xe,
-                         int64_t xe_ld) {
+                         const float* __restrict__ w, float eps, float mult, Residual form,
+                         E* __restrict__ xe, int64_t xe_ld) {
   extern __shared__ __align__(16) float v[];  // [width]
   __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
   const int64_t t = blockIdx.x;
   float* xr = x + t * width;
+  const bool after = form == Residual::kAddNorm;  // the norm is of the sum
   const bool four = width % 4 == 0 && s.part_stride % 4 == 0;
   float ss = 0.f;
   if (four) {
@@ -73,6 +76,11 @@ __global__ void __launch_bounds__(DR_THREADS)
         for (int p = 0; p < s.parts; ++p)
           add4(y, *reinterpret_cast<const float4*>(s.y + p * s.part_stride + t * width + i));
       }
+      if (after) {
+        const float4 r = *reinterpret_cast<const float4*>(xr + i);
+        y.x = fmaf(mult, r.x, y.x), y.y = fmaf(mult, r.y, y.y);
+        y.z = fmaf(mult, r.z, y.z), y.w = fmaf(mult, r.w, y.w);
+      }
       *reinterpret_cast<float4*>(v + i) = y;
       ss += sum_sq4(y);
     }
@@ -87,6 +95,7 @@ __global__ void __launch_bounds__(DR_THREADS)
         y = s.y[t * width + i];
         for (int p = 1; p < s.parts; ++p) y += s.y[p * s.part_stride + t * width + i];
       }
+      if (after) y = fmaf(mult, xr[i], y);
       v[i] = y;
       ss += y * y;
     }
@@ -96,17 +105,22 @@ __global__ void __launch_bounds__(DR_THREADS)
   if (four) {
 #pragma unroll 2
     for (int i = threadIdx.x * 4; i < width; i += DR_THREADS * 4) {
-      float4 r = *reinterpret_cast<const float4*>(xr + i);
       const float4 y = *reinterpret_cast<const float4*>(v + i);
       const float4 k = *reinterpret_cast<const float4*>(w + i);
-      r.x += mult * (y.x * inv * k.x), r.y += mult * (y.y * inv * k.y);
-      r.z += mult * (y.z * inv * k.z), r.w += mult * (y.w * inv * k.w);
+      float4 r;
+      if (after) {
+        r = make_float4(y.x * inv * k.x, y.y * inv * k.y, y.z * inv * k.z, y.w * inv * k.w);
+      } else {
+        r = *reinterpret_cast<const float4*>(xr + i);
+        r.x += mult * (y.x * inv * k.x), r.y += mult * (y.y * inv * k.y);
+        r.z += mult * (y.z * inv * k.z), r.w += mult * (y.w * inv * k.w);
+      }
       *reinterpret_cast<float4*>(xr + i) = r;
       if (xe) store4(xe + t * xe_ld + i, r.x, r.y, r.z, r.w);
     }
   } else {
     for (int i = threadIdx.x; i < width; i += DR_THREADS) {
-      const float r = xr[i] + mult * (v[i] * inv * w[i]);
+      const float n = v[i] * inv * w[i], r = after ? n : xr[i] + mult * n;
       xr[i] = r;
       if (xe) xe[t * xe_ld + i] = to_elem<E>(r);
     }
@@ -242,12 +256,11 @@ __global__ void expert_sum_kernel(const float* __restrict__ ye, const uint32_t* 
 }
 
 // Router and choice, one CTA per RW rows: its warps share out the experts, two at a time
-// (logits = router . x in f32), then one warp per row takes the softmax over all experts, the `top`
-// largest (ties to the lower number) and their shares as weights without renormalising.
+// (logits = router . x + bias in f32), then one warp per row makes the choice (warp_route).
 template <int RW>
 __global__ void __launch_bounds__(DR_THREADS)
     route_kernel(const float* __restrict__ x, int width, const float* __restrict__ router, int ld,
-                 int experts, int top, uint32_t* __restrict__ sel, float* __restrict__ weight,
+                 const float* __restrict__ bias, int experts, int top, RouteWeights form, uint32_t* __restrict__ sel, float* __restrict__ weight,
                  uint32_t* __restrict__ counts, uint32_t* __restrict__ slot, int64_t T) {
   extern __shared__ __align__(16) float sm[];
   pdl_launch_dependents();
@@ -285,13 +298,14 @@ __global__ void __launch_bounds__(DR_THREADS)
     for (int i = 0; i < RW * 2; ++i) {
 #pragma unroll
       for (int o = 16; o; o >>= 1) acc[i] += __shfl_xor_sync(0xFFFFFFFFu, acc[i], o);
-      if (lane == 0 && e0 + i % 2 < experts) l[i / 2 * experts + e0 + i % 2] = acc[i];
+      const int e = e0 + i % 2;
+      if (lane == 0 && e < experts) l[i / 2 * experts + e] = acc[i] + (bias ? bias[e] : 0.f);
     }
   }
   __syncthreads();
   const int64_t t = t0 + warp;
   if (warp >= RW || t >= T) return;
-  warp_route(l + warp * experts, experts, top, lane, sel + t * top, weight + t * top);
+  warp_route(l + warp * experts, experts, top, form, lane, sel + t * top, weight + t * top);
   for (int j = lane; j < top; j += 32)
     slot[t * top + j] = atomicAdd(&counts[sel[t * top + j]], 1u);
 }
@@ -337,6 +351,153 @@ __global__ void __launch_bounds__(DR_THREADS)
   for (int j = threadIdx.x; j < top; j += DR_THREADS) slot[t * top + j] += off[sel[t * top + j]];
 }
 
+// ---- latent attention: what happens to its rows around the products ----
+template <typename E>
+__global__ void __launch_bounds__(DR_THREADS)
+    latent_down_kernel(const LatentStore s, E* __restrict__ cq, int64_t cq_ld) {
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t t = blockIdx.x;
+  if (blockIdx.y == 1) {  // the cache row
+    latent_store_row<E>(s, t, red);
+    return;
+  }
+  const LatentDown& p = s.down;
+  const float* src = p.d + t * p.ld;
+  auto value = [&](int i) {
+    float v = src[i];
+    for (int k = 1; k < p.parts; ++k) v += src[k * p.part_stride + i];
+    return v;
+  };
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < (int)p.q_rank; i += DR_THREADS) {
+    const float v = value(i);
+    ss += v * v;
+  }
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)p.q_rank + p.eps);
+  for (int i = threadIdx.x; i < cq_ld; i += DR_THREADS)
+    cq[t * cq_ld + i] = to_elem<E>(i < (int)p.q_rank ? value(i) * inv * p.q_norm[i] : 0.f);
+}
+
+template <typename E>
+__global__ void __launch_bounds__(DR_THREADS)
+    latent_q_heads_kernel(const LatentAttn a, const LatentQuery q, const uint32_t* __restrict__ rows,
+                          int64_t n, E* __restrict__ out, int ld) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t i = blockIdx.x, t = rows ? rows[i] : i;
+  const float* src = q.q + t * q.ld;
+  for (int k = threadIdx.x; k < (int)a.heads * ld; k += DR_THREADS) {
+    const int h = k / ld, d = k - h * ld;
+    float v = 0.f;
+    if (d < (int)a.dim) {
+      const float* at = src + (int64_t)h * (a.dim + a.rot) + d;
+      v = at[0];
+      for (int p = 1; p < q.parts; ++p) v += at[p * q.part_stride];
+    }
+    out[((int64_t)h * n + i) * ld + d] = to_elem<E>(v);
+  }
+}
+
+__global__ void __launch_bounds__(DR_THREADS)
+    latent_q_rows_kernel(const LatentAttn a, const LatentQuery q,
+                         const uint32_t* __restrict__ positions, bf16* __restrict__ out, int ld,
+                         bf16* __restrict__ out_rot, int rot_ld) {
+  extern __shared__ float2 turn[];  // [rot / 2] (sin, cos)
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  for (int i = threadIdx.x; i < (int)a.rot / 2; i += DR_THREADS)
+    rope_sincos(positions[t], a.freq[i], &turn[i].x, &turn[i].y);
+  pdl_wait();
+  __syncthreads();
+  const float* src = q.q + t * q.ld;
+  const int D = a.dim, RD = a.rot, H = a.heads;
+  auto value = [&](int64_t i) {
+    float v = src[i];
+    for (int p = 1; p < q.parts; ++p) v += src[p * q.part_stride + i];
+    return v;
+  };
+  // two columns at a time (the leading dimensions are even)
+  for (int k = threadIdx.x * 2; k < H * ld; k += DR_THREADS * 2) {
+    const int h = k / ld, d = k - h * ld;
+    const int64_t at = (int64_t)h * (D + RD) + d;
+    const float u = d < D ? value(at) : 0.f, v = d + 1 < D ? value(at + 1) : 0.f;
+    *reinterpret_cast<__nv_bfloat162*>(out + (t * H + h) * ld + d) = __floats2bfloat162_rn(u, v);
+  }
+  for (int k = threadIdx.x * 2; k < H * rot_ld; k += DR_THREADS * 2) {
+    const int h = k / rot_ld, d = k - h * rot_ld;
+    float u = 0.f, v = 0.f;
+    if (d < RD) {
+      const int64_t at = (int64_t)h * (D + RD) + D + d;
+      const float x = value(at), y = value(at + 1);
+      const float2 sc = turn[d / 2];
+      u = x * sc.y - y * sc.x;
+      v = y * sc.y + x * sc.x;
+    }
+    *reinterpret_cast<__nv_bfloat162*>(out_rot + (t * H + h) * rot_ld + d) =
+        __floats2bfloat162_rn(u, v);
+  }
+}
+
+// A warp per cache row.
+__global__ void __launch_bounds__(DR_THREADS)
+    latent_gather_kernel(const KvDenseLayer kv, const RowMap map, const AttnTile* __restrict__ runs,
+                         int n_runs, int R, int RD, bf16* __restrict__ c, int c_ld,
+                         bf16* __restrict__ rot, int rot_ld, int64_t n, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t i = ((int64_t)blockIdx.x * DR_THREADS + threadIdx.x) >> 5;
+  const int lane = threadIdx.x & 31;
+  if (i >= n) return;
+  int r = 0;
+  while (r + 1 < n_runs && i >= runs[r + 1].row0) ++r;
+  const uint32_t j = (uint32_t)(i - runs[r].row0), seq = runs[r].pos0, place = j / kv.block_size;
+  uint32_t block = kv.num_blocks;
+  if (place < map.max_blocks) block = map.tables[(int64_t)seq * map.max_blocks + place];
+  if (block >= kv.num_blocks) {
+    if (lane == 0) atomicOr(status, DEV_BAD_INDEX);
+    block = 0;
+  }
+  const bf16* src = reinterpret_cast<const bf16*>(kv.base) + kv.k_elem(block, 0, j % kv.block_size);
+  if (R % 8 == 0) {
+    for (int d = lane * 8; d < R; d += 256)
+      *reinterpret_cast<uint4*>(c + i * c_ld + d) = *reinterpret_cast<const uint4*>(src + d);
+  } else {
+    for (int d = lane; d < c_ld; d += 32) c[i * c_ld + d] = d < R ? src[d] : to_elem<bf16>(0.f);
+  }
+  for (int d = lane; d < rot_ld; d += 32)
+    rot[i * rot_ld + d] = d < RD ? src[R + d] : to_elem<bf16>(0.f);
+}
+
+// ---- matrix memory: the heads' outputs on the way to the o-projection ----
+template <typename E>
+__global__ void __launch_bounds__(DR_THREADS)
+    head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ gate,
+                          int64_t gate_ld, int parts, int64_t part_stride, int heads, int hd,
+                          const float* __restrict__ w, float eps, E* __restrict__ out,
+                          int64_t out_ld) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = heads * hd;
+  const float *x = o + t * n, *g = gate + t * gate_ld;
+  for (int h = warp; h < heads; h += DR_THREADS / 32) {
+    float ss = 0.f;
+    for (int i = lane; i < hd; i += 32) ss += x[h * hd + i] * x[h * hd + i];
+#pragma unroll
+    for (int s = 16; s; s >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, s);
+    const float inv = 1.0f / sqrtf(ss / (float)hd + eps);
+    for (int i = h * hd + lane; i < (h + 1) * hd; i += 32) {
+      float z = g[i];
+      for (int p = 1; p < parts; ++p) z += g[p * part_stride + i];
+      out[t * out_ld + i] = to_elem<E>(x[i] * inv * w[i] / (1.0f + expf(-z)));
+    }
+  }
+  for (int i = n + threadIdx.x; i < out_ld; i += DR_THREADS) out[t * out_ld + i] = to_elem<E>(0.f);
+}
+
 #define DR_LAUNCH(kern, grid, threads, smem, what, ...)                                          \
   do {                                                                                           \
     const cudaError_t e_ = launch_dependent(ctx, kern, dim3((unsigned)(grid)), dim3(threads),    \
@@ -360,7 +521,7 @@ int32_t launch_embed_scaled(kanso_cuda_ctx* ctx, int32_t compute, const void* em
 
 int32_t launch_residual_norm(kanso_cuda_ctx* ctx, int32_t compute, float* x, int64_t width,
                              const ResidualSource& s, const float* w, float eps, float mult,
-                             void* xe, int64_t xe_ld, int64_t T) {
+                             Residual form, void* xe, int64_t xe_ld, int64_t T) {
   const size_t smem = (size_t)width * 4;
   if (smem > 200 * 1024)
     return fail(ctx, KANSO_ERR_UNSUPPORTED, "residual norm: width %lld", (long long)width);
@@ -371,9 +532,9 @@ int32_t launch_residual_norm(kanso_cuda_ctx* ctx, int32_t compute, float* x, int
   if (st) return st;
   if (compute == KANSO_COMPUTE_BF16)
     DR_LAUNCH(kern_b, T, DR_THREADS, smem, "residual_norm", x, (int)width, s, w, eps, mult,
-              (bf16*)xe, xe_ld);
+              form, (bf16*)xe, xe_ld);
   DR_LAUNCH(kern_f, T, DR_THREADS, smem, "residual_norm", x, (int)width, s, w, eps, mult,
-            (float*)xe, xe_ld);
+            form, (float*)xe, xe_ld);
 }
 
 int32_t launch_expert_sum(kanso_cuda_ctx* ctx, const float* ye, const uint32_t* slot,
@@ -413,7 +574,7 @@ int32_t launch_qk_norm_store(kanso_cuda_ctx* ctx, int32_t compute, const QkvSour
 }
 
 int32_t launch_route(kanso_cuda_ctx* ctx, const float* x, int64_t width, const DenseMat& router,
-                     uint32_t top, uint32_t* sel, float* weight, uint32_t* counts, uint32_t* slot,
+                     const float* bias, uint32_t top, RouteWeights form, uint32_t* sel, float* weight, uint32_t* counts, uint32_t* slot,
                      int64_t T) {
   const int experts = (int)router.rows, ld = (int)router.ld;
   // four rows per CTA where that leaves every SM two of them
@@ -426,7 +587,7 @@ int32_t launch_route(kanso_cuda_ctx* ctx, const float* x, int64_t width, const D
   int32_t st = allow_max_smem(ctx, (const void*)kern);
   if (st) return st;
   DR_LAUNCH(kern, (T + rw - 1) / rw, DR_THREADS, smem, "route", x, (int)width,
-            (const float*)router.w, ld, experts, (int)top, sel, weight, counts, slot, T);
+            (const float*)router.w, ld, bias, experts, (int)top, form, sel, weight, counts, slot, T);
 }
 
 int32_t launch_expert_gather(kanso_cuda_ctx* ctx, int32_t compute, const uint32_t* counts,
@@ -438,6 +599,61 @@ int32_t launch_expert_gather(kanso_cuda_ctx* ctx, int32_t compute, const uint32_
               (int)experts, (int)top, sel, slot, offsets, (const bf16*)xe, ld, (bf16*)xs);
   DR_LAUNCH(expert_gather_kernel<float>, T, DR_THREADS, smem, "expert_gather", counts,
             (int)experts, (int)top, sel, slot, offsets, (const float*)xe, ld, (float*)xs);
+}
+
+std::vector<double> rope_frequencies(uint32_t dims, double base) {
+  std::vector<double> f(dims / 2);
+  for (uint32_t i = 0; i < dims / 2; ++i) f[i] = std::pow(base, -2.0 * i / dims);
+  return f;
+}
+
+int32_t launch_latent_down(kanso_cuda_ctx* ctx, int32_t compute, const LatentStore& s, void* cq,
+                           int64_t T) {
+  const int64_t ld = round_up8(s.down.q_rank);
+  const dim3 grid((unsigned)T, 2);
+  const cudaError_t e =
+      compute == KANSO_COMPUTE_BF16
+          ? launch_dependent(ctx, latent_down_kernel<bf16>, grid, dim3(DR_THREADS), 0, s, (bf16*)cq,
+                             ld)
+          : launch_dependent(ctx, latent_down_kernel<float>, grid, dim3(DR_THREADS), 0, s,
+                             (float*)cq, ld);
+  if (e != cudaSuccess) return cuda_fail(ctx, e, "latent_down");
+  return after_launch(ctx, "latent_down");
+}
+
+int32_t launch_latent_q_heads(kanso_cuda_ctx* ctx, int32_t compute, const LatentAttn& a,
+                              const LatentQuery& q, const uint32_t* rows, int64_t n, void* out) {
+  const int ld = (int)round_up8(a.dim);
+  if (compute == KANSO_COMPUTE_BF16)
+    DR_LAUNCH(latent_q_heads_kernel<bf16>, n, DR_THREADS, 0, "latent_q_heads", a, q, rows, n,
+              (bf16*)out, ld);
+  DR_LAUNCH(latent_q_heads_kernel<float>, n, DR_THREADS, 0, "latent_q_heads", a, q, rows, n,
+            (float*)out, ld);
+}
+
+int32_t launch_latent_q_rows(kanso_cuda_ctx* ctx, const LatentAttn& a, const LatentQuery& q,
+                             const uint32_t* positions, bf16* out, bf16* out_rot, int64_t T) {
+  DR_LAUNCH(latent_q_rows_kernel, T, DR_THREADS, (size_t)a.rot * 4, "latent_q_rows", a, q, positions,
+            out, (int)round_up8(a.dim), out_rot, (int)round_up8(a.rot));
+}
+
+int32_t launch_latent_gather(kanso_cuda_ctx* ctx, const LatentAttn& a, const KvDenseLayer& kv,
+                             const RowMap& map, const AttnTile* runs, uint32_t n_runs, bf16* c,
+                             bf16* rot, int64_t n) {
+  DR_LAUNCH(latent_gather_kernel, (n + DR_THREADS / 32 - 1) / (DR_THREADS / 32), DR_THREADS, 0,
+            "latent_gather", kv, map, runs, (int)n_runs, (int)a.rank, (int)a.rot, c,
+            (int)round_up8(a.rank), rot, (int)round_up8(a.rot), n, ctx->dev_status);
+}
+
+int32_t launch_head_norm_gate(kanso_cuda_ctx* ctx, int32_t compute, const MlstmArgs& a,
+                              const float* w, float eps, void* out, int64_t out_ld, int64_t T) {
+  const int H = a.heads, V = a.vdim;
+  const float* gate = a.y + (int64_t)H * (2 * a.dim + V);
+  if (compute == KANSO_COMPUTE_BF16)
+    DR_LAUNCH(head_norm_gate_kernel<bf16>, T, DR_THREADS, 0, "head_norm_gate", a.out, gate,
+              a.width(), a.parts, a.part_stride, H, V, w, eps, (bf16*)out, out_ld);
+  DR_LAUNCH(head_norm_gate_kernel<float>, T, DR_THREADS, 0, "head_norm_gate", a.out, gate,
+            a.width(), a.parts, a.part_stride, H, V, w, eps, (float*)out, out_ld);
 }
 
 }  // namespace kanso

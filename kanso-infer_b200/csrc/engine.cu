@@ -1,5 +1,6 @@
-// The engine over any model class: cache pages of live requests, ragged steps over them, and
-// greedy generation with continuous batching. Host code only; it drives the model's own step.
+// The engine over any model class: cache pages and state slots of live requests, ragged steps over
+// them, and greedy generation with continuous batching. Host code only; it drives the model's own
+// step. A slot is not cleared when it changes hands: a sequence's first token reads no state.
 #include <algorithm>
 #include <cstring>
 #include <deque>
@@ -12,10 +13,12 @@ using namespace kanso;
 namespace {
 constexpr uint32_t MAX_STEP_TOKENS = 4096;  // rows of one model step (bounds the workspace)
 constexpr uint32_t DEFAULT_STEP_TOKENS = 2048;
+constexpr uint32_t NO_SLOT = 0xFFFFFFFFu;
 
 struct Sequence {
   uint32_t len = 0;         // tokens in the cache
   uint32_t first_live = 0;  // table entries before it have gone back to the pool
+  uint32_t slot = NO_SLOT;  // where its recurrent state lies, from its first step on
   std::vector<uint32_t> table;
 };
 // The next tokens of one sequence in a step.
@@ -31,24 +34,30 @@ struct kanso_cuda_engine {
   kanso_cuda_ctx* ctx = nullptr;
   kanso_cuda_kv* kv = nullptr;
   uint32_t block_size = 16, num_blocks = 0, max_seqs = 0;
-  std::vector<uint32_t> free_blocks;
+  std::vector<uint32_t> free_blocks, free_slots;
   std::unordered_map<uint64_t, Sequence> live;
   uint32_t* d_next = nullptr;  // greedy tokens of a step
   size_t d_next_cap = 0;
-  std::vector<uint32_t> tokens, query_lens, context_lens, tables;  // host image of a step
+  std::vector<uint32_t> tokens, query_lens, context_lens, tables, slots;  // host image of a step
 
   ~kanso_cuda_engine() {
     kanso_cuda_kv_destroy(kv);
     if (d_next) cudaFree(d_next);
   }
 
-  // Pages for `n` more tokens of s; nothing changes when there are too few.
+  // Pages for `n` more tokens of s and a state slot; nothing changes when there are too few.
   int32_t reserve(Sequence* s, uint32_t n) {
     const size_t need = ((uint64_t)s->len + n + block_size - 1) / block_size;
     const size_t more = need > s->table.size() ? need - s->table.size() : 0;
     if (more > free_blocks.size())
       return fail(ctx, KANSO_ERR_SHAPE, "engine: %zu more cache pages needed, %zu free", more,
                   free_blocks.size());
+    if (s->slot == NO_SLOT) {
+      if (free_slots.empty())
+        return fail(ctx, KANSO_ERR_SHAPE, "engine: more than %u live requests", max_seqs);
+      s->slot = free_slots.back();
+      free_slots.pop_back();
+    }
     for (size_t i = 0; i < more; ++i) {
       s->table.push_back(free_blocks.back());
       free_blocks.pop_back();
@@ -57,6 +66,7 @@ struct kanso_cuda_engine {
   }
   void release(Sequence* s) {
     for (size_t i = s->first_live; i < s->table.size(); ++i) free_blocks.push_back(s->table[i]);
+    if (s->slot != NO_SLOT) free_slots.push_back(s->slot);
     *s = Sequence();
   }
   // Gives back the pages that no later token can see.
@@ -75,6 +85,7 @@ struct kanso_cuda_engine {
     tokens.clear();
     query_lens.clear();
     context_lens.clear();
+    slots.clear();
     size_t max_blocks = 1;
     for (const Portion& p : ps) {
       const int32_t st = reserve(p.seq, p.n);
@@ -87,6 +98,7 @@ struct kanso_cuda_engine {
       tokens.insert(tokens.end(), p.tokens, p.tokens + p.n);
       query_lens.push_back(p.n);
       context_lens.push_back(p.seq->len + p.n);
+      slots.push_back(p.seq->slot);
       std::copy(p.seq->table.begin(), p.seq->table.end(), tables.begin() + i * max_blocks);
     }
     StepBatch b;
@@ -97,6 +109,7 @@ struct kanso_cuda_engine {
     b.query_lens = query_lens.data();
     b.context_lens = context_lens.data();
     b.tables = tables.data();
+    b.state_slots = slots.data();
     b.want = want.data();
     b.n_want = (uint32_t)want.size();
     const int32_t st = run_step(model, kv, b);
@@ -125,12 +138,13 @@ int32_t kanso_cuda_engine_create(kanso_cuda_model* m, uint32_t max_tokens, uint3
   e->max_seqs = max_seqs;
   // every request may leave its last page partly filled, and its first one partly retired
   e->num_blocks = (max_tokens + e->block_size - 1) / e->block_size + 2 * max_seqs;
-  const int32_t st = m->create_pool(e->num_blocks, &e->kv);
+  const int32_t st = m->create_pool(e->num_blocks, max_seqs, &e->kv);
   if (st) {
     delete e;
     return st;
   }
   for (uint32_t b = e->num_blocks; b-- > 0;) e->free_blocks.push_back(b);
+  for (uint32_t s = max_seqs; s-- > 0;) e->free_slots.push_back(s);
   *out = e;
   return KANSO_OK;
 }

@@ -35,6 +35,21 @@ struct GemmDenseArgs {
   int64_t T;
   int groups, rows, k_steps, steps_per_split;
   int* status;
+  const float* bias;
+  int64_t group_step;
+  const uint32_t* row_list;
+  int relu2, elem, n_end;  // n_end: columns that are written
+
+  __device__ __forceinline__ float finish(float v, int n) const {
+    if (bias && n < rows && blockIdx.z == 0) v += bias[n];
+    return relu2 ? relu_squared(v) : v;
+  }
+  // Element offset of a result row.
+  __device__ __forceinline__ int64_t row_at(int64_t row, int group) const {
+    if (!group_step) return row * out_ld;
+    const int64_t r = row - group * (T / groups);
+    return (row_list ? row_list[r] : r) * out_ld + group * group_step;
+  }
 };
 
 // The (group, first row, end of the group) of tile `tile`; one warp. false: past the last tile.
@@ -42,10 +57,11 @@ __device__ __forceinline__ bool find_tile(const uint32_t* offsets, int groups, i
                                           int tile, int lane, int* group, int64_t* first,
                                           int64_t* end) {
   if (!offsets) {
-    *group = 0;
-    *first = (int64_t)tile * nt;
-    *end = T;
-    return *first < T;
+    const int64_t per = T / groups, tiles = (per + nt - 1) / nt;
+    *group = (int)(tile / tiles);
+    *first = *group * per + tile % tiles * nt;
+    *end = (*group + 1) * per;
+    return *group < groups;
   }
   int before = 0;
   for (int g0 = 0; g0 < groups; g0 += 32) {
@@ -209,10 +225,18 @@ __global__ void __launch_bounds__(GD_THREADS)
           if (n < a.out_ld)
             static_cast<bf16*>(a.out)[row * a.out_ld + n] = to_elem<bf16>(silu(g) * u);
         } else {
-          float* o = static_cast<float*>(a.out) + (int64_t)blockIdx.z * a.part_stride +
-                     row * a.out_ld;
-          if (n < a.rows) o[n] = __uint_as_float(r0[j]);
-          if (DUAL && n + 128 < a.rows) o[n + 128] = __uint_as_float(r1[j]);
+          const int64_t at = (int64_t)blockIdx.z * a.part_stride + a.row_at(row, tile_group);
+          const float v0 = a.finish(__uint_as_float(r0[j]), n);
+          const float v1 = DUAL ? a.finish(__uint_as_float(r1[j]), n + 128) : 0.f;
+          if (a.elem) {
+            bf16* o = static_cast<bf16*>(a.out) + at;
+            if (n < a.n_end) o[n] = to_elem<bf16>(v0);
+            if (DUAL && n + 128 < a.n_end) o[n + 128] = to_elem<bf16>(v1);
+          } else {
+            float* o = static_cast<float*>(a.out) + at;
+            if (n < a.n_end) o[n] = v0;
+            if (DUAL && n + 128 < a.n_end) o[n + 128] = v1;
+          }
         }
       }
     }
@@ -295,9 +319,9 @@ __global__ void __launch_bounds__(256)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int n = n0 + tx + 16 * i;
-      if (n < (ACT ? a.out_ld : a.rows))
-        static_cast<float*>(a.out)[row * a.out_ld + n] =
-            ACT ? silu(acc[m][i]) * acu[m][i] : acc[m][i];
+      if (n < (ACT ? a.out_ld : a.n_end))
+        static_cast<float*>(a.out)[a.row_at(row, tile_group) + n] =
+            ACT ? silu(acc[m][i]) * acu[m][i] : a.finish(acc[m][i], n);
     }
   }
 }
@@ -346,8 +370,8 @@ static int32_t gd_launch(kanso_cuda_ctx* ctx, dim3 grid, const CUtensorMap& wm,
 
 // Tiles that cover the rows: exact for one group, the most there can be for several.
 static int64_t tiles_of(const GemmRows& r, int nt) {
-  const int64_t t = (r.T + nt - 1) / nt;
-  return r.offsets ? std::min<int64_t>(t + r.groups - 1, r.T) : t;
+  if (!r.offsets) return r.groups * ((r.T / r.groups + nt - 1) / nt);
+  return std::min<int64_t>((r.T + nt - 1) / nt + r.groups - 1, r.T);
 }
 static int pick_nt(const GemmRows& r) {
   const int64_t per = (r.T + r.groups - 1) / r.groups;
@@ -355,12 +379,15 @@ static int pick_nt(const GemmRows& r) {
   return aim <= 16 ? 16 : aim <= 32 ? 32 : aim <= 64 ? 64 : 128;
 }
 
-int32_t launch_gemm(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat& w, const void* x,
-                    float* y, int64_t y_ld, const GemmRows& r, int max_splits, int* splits,
-                    int64_t part_stride) {
+int32_t launch_gemm(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat& w, const void* x, void* y,
+                    int64_t y_ld, const GemmRows& r, int max_splits, int* splits,
+                    int64_t part_stride, const GemmOut& o) {
   *splits = 1;
+  if (o.relu2 || o.elem) max_splits = 1;
+  // pad columns of a result in element type belong to it unless the next group lies behind it
+  const int n_end = (int)(o.elem && !o.group_step ? std::max<int64_t>(y_ld, w.rows) : w.rows);
   GemmDenseArgs a = {y, y_ld, part_stride, r.offsets, r.T, r.groups, (int)w.rows, 0, 0,
-                     ctx->dev_status};
+                     ctx->dev_status, o.bias, o.group_step, o.rows, o.relu2, o.elem, n_end};
   if (compute == KANSO_COMPUTE_F32) {
     const dim3 grid((unsigned)((w.rows + GF_TILE - 1) / GF_TILE), (unsigned)tiles_of(r, GF_TILE));
     const cudaError_t e =
@@ -402,7 +429,7 @@ int32_t launch_gemm_gate_up(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat
                             const DenseMat& up, const void* x, void* act, int64_t act_ld,
                             const GemmRows& r) {
   GemmDenseArgs a = {act, act_ld, 0, r.offsets, r.T, r.groups, (int)gate.rows, 0, 0,
-                     ctx->dev_status};
+                     ctx->dev_status, nullptr, 0, nullptr, 0, 0, 0};
   if (compute == KANSO_COMPUTE_F32) {
     const dim3 grid((unsigned)((gate.rows + GF_TILE - 1) / GF_TILE),
                     (unsigned)tiles_of(r, GF_TILE));

@@ -11,7 +11,8 @@
 // Three kernels use that core: the plain product (with the residual step in front of it where the
 // caller asks, so that a layer needs no norm launch), the experts' gate and up product with the
 // routing decision in front of it, and the experts' down product, whose columns are the chosen
-// experts' one after the other.
+// experts' one after the other. A matrix of several groups (one per head) takes an input of its own
+// for each.
 #include <cmath>
 
 #include "dense.cuh"
@@ -120,7 +121,31 @@ struct GemvArgs {
   GemvSource s;
   float* out;
   int64_t out_ld;
+  GemvOut o;
+  int store_ctas;  // CTAs in front of the product's that store the step's cache rows
+  LatentStore store;
 };
+
+// Each head over its own root mean square, weight and gate (GemvSource::gate): a warp per head.
+__device__ __forceinline__ void gate_source(const GemvSource& s, const float* x, const float* gate,
+                                            int cols, int ld, float* xt) {
+  const int hd = cols / s.heads, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int h = warp; h < s.heads; h += GV_WARPS) {
+    float ss = 0.f;
+    for (int i = lane; i < hd; i += 32) {
+      const float v = x[h * hd + i];
+      ss += v * v;
+    }
+#pragma unroll
+    for (int o = 16; o; o >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, o);
+    const float inv = 1.0f / sqrtf(ss / (float)hd + s.eps);
+    for (int i = h * hd + lane; i < (h + 1) * hd; i += 32) {
+      float g = gate[i];
+      for (int p = 1; p < s.parts; ++p) g += gate[p * s.part_stride + i];
+      xt[xs_index(i, ld)] = x[i] * inv * s.norm_w[i] / (1.0f + expf(-g));
+    }
+  }
+}
 
 // The residual step for the rows of this CTA, into shared memory (and to x_out by one CTA).
 template <int TT>
@@ -129,12 +154,20 @@ __device__ __forceinline__ void norm_source(const GemvSource& s, int cols, int l
   for (int t = 0; t < nt; ++t) {
     const int64_t r = s.row_index ? s.row_index[t0 + t] : t0 + t;
     const float* y = s.y + r * cols;
+    const float* x = s.x + r * (s.x_ld ? s.x_ld : cols) + blockIdx.z * s.x_group;
     float* xt = xs + t * ld;
+    const bool after = s.form == Residual::kAddNorm;
+    if (s.gate) {
+      gate_source(s, x, s.gate + r * s.gate_ld, cols, ld, xt);
+      for (int i = cols + threadIdx.x; i < ld; i += GV_THREADS) xt[xs_index(i, ld)] = 0.f;
+      continue;
+    }
     float ss = 0.f;
     if (s.y) {
       for (int i = threadIdx.x; i < cols; i += GV_THREADS) {
         float v = y[i];
         for (int p = 1; p < s.parts; ++p) v += y[p * s.part_stride + i];
+        if (after) v = fmaf(s.mult, x[i], v);
         xt[xs_index(i, ld)] = v;
         ss += v * v;
       }
@@ -143,8 +176,13 @@ __device__ __forceinline__ void norm_source(const GemvSource& s, int cols, int l
     const float inv = s.y ? 1.0f / sqrtf(ss / (float)cols + s.eps) : 0.f;
     float s2 = 0.f;
     for (int i = threadIdx.x; i < cols; i += GV_THREADS) {
-      float v = s.x[r * cols + i];
-      if (s.y) v += s.mult * (xt[xs_index(i, ld)] * inv * s.norm_w[i]);
+      float v;
+      if (s.y && after) {
+        v = xt[xs_index(i, ld)] * inv * s.norm_w[i];
+      } else {
+        v = x[i];
+        if (s.y) v += s.mult * (xt[xs_index(i, ld)] * inv * s.norm_w[i]);
+      }
       xt[xs_index(i, ld)] = v;
       if (writer && s.x_out) s.x_out[r * cols + i] = v;
       s2 += v * v;
@@ -169,7 +207,15 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_dense_kernel(const GemvArgs a
   const int gpc = GV_WARPS / a.ks, sub = warp % a.ks, chunks = a.ld / 8;
   const int t0 = blockIdx.y * TT, nt = min(TT, a.T - t0);
   const int groups = (a.rows + GV_ROWS - 1) / GV_ROWS;
-  const E* w = static_cast<const E*>(a.w);
+  if ((int)blockIdx.x < a.store_ctas) {
+    pdl_launch_dependents();
+    pdl_wait();
+    if (blockIdx.y == 0 && blockIdx.z == 0) latent_store_row<E>(a.store, blockIdx.x, red);
+    return;
+  }
+  const int cta = blockIdx.x - a.store_ctas, ctas = gridDim.x - a.store_ctas;
+  const E* w = static_cast<const E*>(a.w) + (int64_t)blockIdx.z * a.rows * a.ld;
+  float* out = a.out + blockIdx.z * a.o.group_step;
   const int c0 = sub * 32 + lane, step = a.ks * 32;
   const E* row[GV_ROWS];
   RawOf<E> cur[GV_ROWS];
@@ -180,22 +226,24 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_dense_kernel(const GemvArgs a
       if (c0 < chunks) cur[r] = load_raw_once(row[r] + (size_t)c0 * 8);
     }
   };
-  int base = blockIdx.x * gpc;
+  int base = cta * gpc;
   open_group(base + warp / a.ks);  // weights depend on nothing that runs before this kernel
   pdl_launch_dependents();
   pdl_wait();
-  norm_source<TT>(a.s, a.cols, a.ld, t0, nt, blockIdx.x == 0, xs, red);
+  norm_source<TT>(a.s, a.cols, a.ld, t0, nt, cta == 0 && blockIdx.z == 0, xs, red);
   __syncthreads();
   while (true) {
     float acc[GV_ROWS * TT];
 #pragma unroll
     for (int i = 0; i < GV_ROWS * TT; ++i) acc[i] = 0.f;
     dot_rows<E, TT>(row, cur, c0, step, chunks, xs, a.ld, acc);
-    const int nbase = base + gridDim.x * gpc;
+    const int nbase = base + ctas * gpc;
     if (nbase < groups) open_group(nbase + warp / a.ks);
     finish_rows<GV_ROWS * TT>(acc, a.ks, red, [&](int grp, int idx, float v) {
       const int n = (base + grp) * GV_ROWS + idx / TT, t = idx % TT;
-      if (n < a.rows && t < nt) a.out[(int64_t)(t0 + t) * a.out_ld + n] = v;
+      if (n >= a.rows || t >= nt) return;
+      if (a.o.bias) v += a.o.bias[n];
+      out[(int64_t)(t0 + t) * a.out_ld + n] = a.o.relu2 ? relu_squared(v) : v;
     });
     if (nbase >= groups) break;
     base = nbase;
@@ -205,14 +253,16 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_dense_kernel(const GemvArgs a
 struct GateUpArgs {
   const void *gate, *up;
   int ff, cols, ld, ff_ld, ks, top, experts;
+  RouteWeights form;
   const float* x;
   const float* logits;
   float* act;
   uint32_t* sel;
 };
 
-// Two gate rows and the two up rows beside them per warp step; blockIdx.y = row * top + place.
-template <typename E>
+// Two gate rows and the two up rows beside them per warp step, without a gate four up rows;
+// blockIdx.y = row * top + place.
+template <typename E, bool GATED>
 __global__ void __launch_bounds__(GV_THREADS) gemv_gate_up_kernel(const GateUpArgs a) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[GV_WARPS * GV_ROWS];
@@ -229,39 +279,39 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_gate_up_kernel(const GateUpAr
   for (int i = threadIdx.x; i < a.ld; i += GV_THREADS)
     xs[xs_index(i, a.ld)] = i < a.cols ? a.x[(int64_t)t * a.cols + i] : 0.f;
   __syncthreads();
-  if (warp == 0) warp_route(lg, a.experts, a.top, lane, sel, wt);
+  if (warp == 0) warp_route(lg, a.experts, a.top, a.form, lane, sel, wt);
   __syncthreads();
   if (blockIdx.x == 0 && threadIdx.x == 0) a.sel[blockIdx.y] = sel[place];
   const float weight = wt[place];
   const int64_t ebase = (int64_t)sel[place] * a.ff;
   const int gpc = GV_WARPS / a.ks, sub = warp % a.ks, chunks = a.ld / 8;
-  const int c0 = sub * 32 + lane, groups = (a.ff + 1) / 2;
+  constexpr int PER = GATED ? 2 : 4;  // results per warp step
+  const int c0 = sub * 32 + lane, groups = (a.ff + PER - 1) / PER;
   for (int base = blockIdx.x * gpc; base < groups; base += gridDim.x * gpc) {
-    const int f0 = min(base + warp / a.ks, groups - 1) * 2, f1 = min(f0 + 1, a.ff - 1);
-    const E* row[GV_ROWS] = {static_cast<const E*>(a.gate) + (ebase + f0) * a.ld,
-                             static_cast<const E*>(a.gate) + (ebase + f1) * a.ld,
-                             static_cast<const E*>(a.up) + (ebase + f0) * a.ld,
-                             static_cast<const E*>(a.up) + (ebase + f1) * a.ld};
+    const int f0 = min(base + warp / a.ks, groups - 1) * PER;
+    const E* row[GV_ROWS];
     RawOf<E> cur[GV_ROWS];
-    if (c0 < chunks) {
 #pragma unroll
-      for (int r = 0; r < GV_ROWS; ++r) cur[r] = load_raw_once(row[r] + (size_t)c0 * 8);
+    for (int r = 0; r < GV_ROWS; ++r) {
+      const E* m = static_cast<const E*>(GATED && r < 2 ? a.gate : a.up);
+      row[r] = m + (ebase + min(f0 + (GATED ? r & 1 : r), a.ff - 1)) * a.ld;
+      if (c0 < chunks) cur[r] = load_raw_once(row[r] + (size_t)c0 * 8);
     }
     float acc[GV_ROWS] = {0.f, 0.f, 0.f, 0.f};
     dot_rows<E, 1>(row, cur, c0, a.ks * 32, chunks, xs, a.ld, acc);
     const float s = warp_sum_scatter<GV_ROWS>(acc, lane);  // lane / 8 = row of the four
     if (lane % 8 == 0) red[warp * GV_ROWS + lane / 8] = s;
     __syncthreads();
-    if (threadIdx.x < gpc * 2) {
-      const int grp = threadIdx.x / 2, f = threadIdx.x % 2;
+    if (threadIdx.x < gpc * PER) {
+      const int grp = threadIdx.x / PER, f = threadIdx.x % PER;
       float g = 0.f, u = 0.f;
       for (int k = 0; k < a.ks; ++k) {
         g += red[(grp * a.ks + k) * GV_ROWS + f];
-        u += red[(grp * a.ks + k) * GV_ROWS + 2 + f];
+        if (GATED) u += red[(grp * a.ks + k) * GV_ROWS + 2 + f];
       }
-      const int n = (base + grp) * 2 + f;
+      const int n = (base + grp) * PER + f;
       if (base + grp < groups && n < a.ff)
-        a.act[(int64_t)blockIdx.y * a.ff_ld + n] = weight * (silu(g) * u);
+        a.act[(int64_t)blockIdx.y * a.ff_ld + n] = weight * (GATED ? silu(g) * u : relu_squared(g));
     }
     __syncthreads();
   }
@@ -366,16 +416,20 @@ static int32_t gemv_launch(kanso_cuda_ctx* ctx, const GemvArgs& a, dim3 grid, si
 }
 
 int32_t launch_gemv(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat& w, const GemvSource& s,
-                    float* out, int64_t out_ld, int T) {
+                    float* out, int64_t out_ld, int T, const GemvOut& o, const LatentStore* store) {
   int tt = 1;
   while (tt < T && tt < GEMV_MAX_T && (int64_t)tt * 2 * w.ld * 4 <= 128 * 1024) tt *= 2;
   const size_t smem = (size_t)tt * w.ld * 4;
   if (smem > (size_t)GEMV_MAX_COLS * 4)
     return fail(ctx, KANSO_ERR_UNSUPPORTED, "dense product: %lld columns", (long long)w.cols);
   const int64_t groups = (w.rows + GV_ROWS - 1) / GV_ROWS, copies = (T + tt - 1) / tt;
-  GemvArgs a = {w.w, (int)w.rows, (int)w.cols, (int)w.ld, pick_ks(ctx, groups, copies, w.ld / 8),
-                T, s, out, out_ld};
-  const dim3 grid(gv_grid(ctx, groups, a.ks, copies), (unsigned)copies);
+  const int64_t all = copies * w.groups;
+  if (w.groups > 65535)
+    return fail(ctx, KANSO_ERR_UNSUPPORTED, "dense product: %lld groups", (long long)w.groups);
+  GemvArgs a = {w.w, (int)w.rows, (int)w.cols, (int)w.ld, pick_ks(ctx, groups, all, w.ld / 8),
+                T, s, out, out_ld, o, store ? T : 0, store ? *store : LatentStore()};
+  const dim3 grid(gv_grid(ctx, groups, a.ks, all) + a.store_ctas, (unsigned)copies,
+                  (unsigned)w.groups);
   if (compute == KANSO_COMPUTE_BF16) {
     switch (tt) {
       case 1: return gemv_launch<bf16, 1>(ctx, a, grid, smem);
@@ -388,19 +442,22 @@ int32_t launch_gemv(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat& w, con
   }
 }
 
-int32_t launch_gemv_gate_up(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat& gate,
+int32_t launch_gemv_gate_up(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat* gate,
                             const DenseMat& up, const float* x, const float* router_logits,
-                            uint32_t experts, uint32_t top, float* act, uint32_t* sel, int T) {
-  const int64_t groups = (gate.rows + 1) / 2, copies = (int64_t)T * top;
-  GateUpArgs a = {gate.w, up.w, (int)gate.rows, (int)gate.cols, (int)gate.ld,
-                  (int)round_up8(gate.rows), pick_ks(ctx, groups, copies, gate.ld / 8), (int)top,
-                  (int)experts, x, router_logits, act, sel};
+                            uint32_t experts, uint32_t top, RouteWeights form, float* act,
+                            uint32_t* sel, int T) {
+  const int64_t per = gate ? 2 : 4, groups = (up.rows + per - 1) / per, copies = (int64_t)T * top;
+  GateUpArgs a = {gate ? gate->w : nullptr, up.w, (int)up.rows, (int)up.cols, (int)up.ld,
+                  (int)round_up8(up.rows), pick_ks(ctx, groups, copies, up.ld / 8), (int)top,
+                  (int)experts, form, x, router_logits, act, sel};
   const dim3 grid(gv_grid(ctx, groups, a.ks, copies), (unsigned)copies);
-  const size_t smem = ((size_t)gate.ld + experts + 2 * top) * 4;
+  const size_t smem = ((size_t)up.ld + experts + 2 * top) * 4;
   if (smem > (size_t)GEMV_MAX_COLS * 4)
     return fail(ctx, KANSO_ERR_UNSUPPORTED, "expert product: %lld columns, %u experts",
-                (long long)gate.cols, experts);
-  auto kern = compute == KANSO_COMPUTE_BF16 ? gemv_gate_up_kernel<bf16> : gemv_gate_up_kernel<float>;
+                (long long)up.cols, experts);
+  const bool b16 = compute == KANSO_COMPUTE_BF16;
+  auto kern = gate ? (b16 ? gemv_gate_up_kernel<bf16, true> : gemv_gate_up_kernel<float, true>)
+                   : (b16 ? gemv_gate_up_kernel<bf16, false> : gemv_gate_up_kernel<float, false>);
   int32_t st = allow_max_smem(ctx, (const void*)kern);
   if (st) return st;
   const cudaError_t e = launch_dependent(ctx, kern, grid, dim3(GV_THREADS), smem, a);

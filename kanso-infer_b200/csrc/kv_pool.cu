@@ -145,11 +145,36 @@ int32_t kanso_cuda_kv_create_dense(kanso_cuda_ctx* ctx, uint32_t num_layers,
   if (!out || !kv_heads || !k_dim || !v_dim)
     return fail(ctx, KANSO_ERR_CONFIG, "kv_create_dense: NULL argument");
   *out = nullptr;
+  std::vector<kanso_kv_layer> l(num_layers);
+  for (uint32_t i = 0; i < num_layers; ++i) {
+    if (!kv_heads[i] || !k_dim[i] || !v_dim[i])
+      return fail(ctx, KANSO_ERR_CONFIG, "kv_create_dense: layer %u has a zero size", i);
+    l[i] = {kv_heads[i], k_dim[i], v_dim[i], 0, 0, 0};
+  }
+  return kanso_cuda_kv_create_layers(ctx, num_layers, l.data(), num_blocks, block_size, kv_type, 0,
+                                     out);
+}
+
+int32_t kanso_cuda_kv_create_layers(kanso_cuda_ctx* ctx, uint32_t num_layers,
+                                    const kanso_kv_layer* layers, uint32_t num_blocks,
+                                    uint32_t block_size, int32_t kv_type, uint32_t num_slots,
+                                    kanso_cuda_kv** out) {
+  if (!ctx) return fail(nullptr, KANSO_ERR_CONFIG, "kv_create_layers: ctx is NULL");
+  if (!out || !layers) return fail(ctx, KANSO_ERR_CONFIG, "kv_create_layers: NULL argument");
+  *out = nullptr;
   if (kv_type != KANSO_KV_BF16 && kv_type != KANSO_KV_F32)
-    return fail(ctx, KANSO_ERR_CONFIG, "kv_create_dense: kv type %d (expected bf16 or f32)",
+    return fail(ctx, KANSO_ERR_CONFIG, "kv_create_layers: kv type %d (expected bf16 or f32)",
                 kv_type);
   if (!num_layers || !num_blocks || !block_size)
-    return fail(ctx, KANSO_ERR_CONFIG, "kv_create_dense: every dimension must be non-zero");
+    return fail(ctx, KANSO_ERR_CONFIG, "kv_create_layers: every dimension must be non-zero");
+  for (uint32_t i = 0; i < num_layers; ++i) {
+    const kanso_kv_layer& l = layers[i];
+    if ((l.kv_heads && !l.k_dim) || (l.state_heads && (!l.state_dim || !l.state_vdim)))
+      return fail(ctx, KANSO_ERR_CONFIG, "kv_create_layers: layer %u has a zero size", i);
+    if (l.state_heads && !num_slots)
+      return fail(ctx, KANSO_ERR_CONFIG, "kv_create_layers: layer %u keeps a state, there are no "
+                                         "slots", i);
+  }
   const size_t es = kv_type == KANSO_KV_BF16 ? 2 : 4;
   auto* kv = new kanso_cuda_kv;
   kv->ctx = ctx;
@@ -157,44 +182,62 @@ int32_t kanso_cuda_kv_create_dense(kanso_cuda_ctx* ctx, uint32_t num_layers,
   kv->num_blocks = num_blocks;
   kv->block_size = block_size;
   kv->kv_type = kv_type;
+  kv->num_slots = num_slots;
   kv->dense.resize(num_layers);
+  kv->state.resize(num_layers);
   size_t bytes = 0;
-  std::vector<size_t> at(num_layers);
-  for (uint32_t l = 0; l < num_layers; ++l) {
-    KvDenseLayer& d = kv->dense[l];
-    if (!kv_heads[l] || !k_dim[l] || !v_dim[l]) {
-      delete kv;
-      return fail(ctx, KANSO_ERR_CONFIG, "kv_create_dense: layer %u has a zero size", l);
-    }
-    d.kv_heads = kv_heads[l];
-    d.k_dim = k_dim[l];
-    d.v_dim = v_dim[l];
-    d.k_ld = (k_dim[l] + 7u) & ~7u;
-    d.v_ld = (v_dim[l] + 7u) & ~7u;
+  std::vector<size_t> at(num_layers), state_at(num_layers);
+  auto room = [&](size_t n) {
+    const size_t p = bytes;
+    bytes += (n + 255) & ~(size_t)255;
+    return p;
+  };
+  for (uint32_t i = 0; i < num_layers; ++i) {
+    const kanso_kv_layer& l = layers[i];
+    KvDenseLayer& d = kv->dense[i];
+    d.kv_heads = l.kv_heads;
+    d.k_dim = l.k_dim;
+    d.v_dim = l.v_dim;
+    d.k_ld = (l.k_dim + 7u) & ~7u;
+    d.v_ld = (l.v_dim + 7u) & ~7u;
     d.block_size = block_size;
     d.num_blocks = num_blocks;
     d.rec_elems = block_size * (d.k_ld + d.v_ld);
-    at[l] = bytes;
-    bytes += ((size_t)num_blocks * d.kv_heads * d.rec_elems * es + 255) & ~(size_t)255;
+    at[i] = room((size_t)num_blocks * d.kv_heads * d.rec_elems * es);
+    KvStateLayer& s = kv->state[i];
+    s.heads = l.state_heads;
+    s.dim = l.state_dim;
+    s.vdim = l.state_vdim;
+    state_at[i] = room(s.heads ? s.slot_floats() * num_slots * 4 : 0);
   }
-  cudaError_t e = cudaMalloc((void**)&kv->pool, bytes);
+  cudaError_t e = cudaMalloc((void**)&kv->pool, bytes + 256);
   if (e != cudaSuccess) {
     delete kv;
     cudaGetLastError();
-    return fail(ctx, KANSO_ERR_CONFIG, "kv_create_dense: cannot allocate %zu bytes of KV pool: %s",
+    return fail(ctx, KANSO_ERR_CONFIG, "kv_create_layers: cannot allocate %zu bytes of KV pool: %s",
                 bytes, cudaGetErrorString(e));
   }
   kv->pool_bytes = bytes;
-  for (uint32_t l = 0; l < num_layers; ++l) kv->dense[l].base = kv->pool + at[l];
+  for (uint32_t i = 0; i < num_layers; ++i) {
+    kv->dense[i].base = kv->pool + at[i];
+    kv->state[i].base = reinterpret_cast<float*>(kv->pool + state_at[i]);
+  }
   // masked keys are multiplied by zero: no row may hold a NaN
   e = cudaMemsetAsync(kv->pool, 0, bytes, ctx->stream);
   if (e != cudaSuccess) {
     cudaFree(kv->pool);
     delete kv;
-    return cuda_fail(ctx, e, "kv_create_dense: clear");
+    return cuda_fail(ctx, e, "kv_create_layers: clear");
   }
   *out = kv;
   return KANSO_OK;
+}
+
+uint64_t kanso_cuda_kv_state_bytes(const kanso_cuda_kv* kv) {
+  uint64_t n = 0;
+  if (kv)
+    for (const KvStateLayer& s : kv->state) n += s.heads ? s.slot_floats() * 4 : 0;
+  return n;
 }
 
 int32_t kanso_cuda_kv_destroy(kanso_cuda_kv* kv) {
@@ -235,10 +278,11 @@ int32_t kanso_cuda_kv_reset_block(kanso_cuda_ctx* ctx, kanso_cuda_kv* kv, uint32
   if (!kv->dense.empty()) {
     const size_t es = kv->kv_type == KANSO_KV_BF16 ? 2 : 4;
     for (const KvDenseLayer& d : kv->dense)
-      KANSO_CUDA_TRY(ctx,
-                     cudaMemsetAsync(d.base + d.k_elem(block, 0, 0) * es, 0,
-                                     (size_t)d.kv_heads * d.rec_elems * es, ctx->stream),
-                     "kv_reset_block");
+      if (d.kv_heads)
+        KANSO_CUDA_TRY(ctx,
+                       cudaMemsetAsync(d.base + d.k_elem(block, 0, 0) * es, 0,
+                                       (size_t)d.kv_heads * d.rec_elems * es, ctx->stream),
+                       "kv_reset_block");
     return KANSO_OK;
   }
   KvGeom g = kv_geom(kv);

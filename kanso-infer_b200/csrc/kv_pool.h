@@ -13,7 +13,10 @@
 //
 // An unquantised pool (bf16 or f32 rows; `dense` not empty) keeps, per layer, one record per
 // (block, kv head): [ K rows block_size x k_ld ][ V rows block_size x v_ld ], row lengths rounded
-// up to 8 elements with zeros behind. Layers may differ in heads and in key and value size.
+// up to 8 elements with zeros behind. Layers may differ in heads and in key and value size. A layer
+// of latent attention has one head whose row is the latent and the rotated key part behind it,
+// and no value rows. A recurrent layer has no rows; it keeps one state per sequence instead, in the
+// slot that the host gives to the sequence (KvStateLayer).
 #pragma once
 #include "ctx.h"
 
@@ -32,6 +35,26 @@ struct KvDenseLayer {
            (size_t)off * v_ld;
   }
 };
+
+// The recurrent state of one layer, f32, per (slot, head, tile of 32 value columns) one record
+//
+//   [ S dim x 32 ][ n dim, rounded up to 4 ][ m, 3 unused ]
+//
+// with its own copy of n and of the maximum m, so that the tiles of a head need nothing of one
+// another. The state before position 0 is never read.
+struct KvStateLayer {
+  static constexpr uint32_t kCols = 32;
+  float* base = nullptr;
+  uint32_t heads = 0, dim = 0, vdim = 0;
+  __host__ __device__ uint32_t tiles() const { return (vdim + kCols - 1) / kCols; }
+  __host__ __device__ uint32_t n_at() const { return dim * kCols; }
+  __host__ __device__ uint32_t m_at() const { return n_at() + ((dim + 3u) & ~3u); }
+  __host__ __device__ uint32_t rec() const { return m_at() + 4; }
+  __host__ __device__ size_t slot_floats() const { return (size_t)heads * tiles() * rec(); }
+  __host__ __device__ float* at(uint32_t slot, uint32_t head, uint32_t tile) const {
+    return base + slot * slot_floats() + (size_t)(head * tiles() + tile) * rec();
+  }
+};
 }  // namespace kanso
 
 struct kanso_cuda_kv {
@@ -42,6 +65,9 @@ struct kanso_cuda_kv {
   size_t pool_bytes = 0;
   // one entry per layer of an unquantised pool; kv_heads and head_dim are then 0
   std::vector<kanso::KvDenseLayer> dense;
+  // the same length; heads 0: the layer has no state
+  std::vector<kanso::KvStateLayer> state;
+  uint32_t num_slots = 0;
 };
 
 namespace kanso {

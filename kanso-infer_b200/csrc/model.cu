@@ -68,12 +68,13 @@ struct LlamaModel final : kanso_cuda_model {
   uint32_t block_size() const override { return cfg.block_size ? cfg.block_size : 16; }
   uint32_t max_positions() const override { return cfg.max_seq_len; }
   uint32_t max_query_len() const override { return 1; }  // its step is the decode step
-  int32_t create_pool(uint32_t num_blocks, kanso_cuda_kv** out) override;
+  int32_t create_pool(uint32_t num_blocks, uint32_t num_slots, kanso_cuda_kv** out) override;
   int32_t check_pool(const kanso_cuda_kv* kv) override;
   int32_t decode_device(kanso_cuda_kv* kv, const uint32_t* tokens, const uint32_t* positions,
                         const uint32_t* slots, const uint32_t* tables,
-                        const uint32_t* context_lens, uint32_t B, uint32_t max_blocks,
-                        uint32_t max_ctx, int32_t act_mode, float* logits_dev) override;
+                        const uint32_t* context_lens, const uint32_t* state_slots, uint32_t B,
+                        uint32_t max_blocks, uint32_t max_ctx, int32_t act_mode,
+                        float* logits_dev) override;
   int32_t forward(kanso_cuda_kv* kv, const kanso::StepBatch& b, float* logits_dev) override;
 };
 
@@ -277,7 +278,7 @@ LlamaModel::~LlamaModel() {
   if (rope_sin) cudaFree(rope_sin);
 }
 
-int32_t LlamaModel::create_pool(uint32_t num_blocks, kanso_cuda_kv** out) {
+int32_t LlamaModel::create_pool(uint32_t num_blocks, uint32_t, kanso_cuda_kv** out) {
   return kanso_cuda_kv_create(ctx, cfg.num_hidden_layers, num_blocks, block_size(),
                               cfg.num_key_value_heads, cfg.hidden_size / cfg.num_attention_heads,
                               KANSO_KV_INT8, out);
@@ -316,7 +317,7 @@ int32_t LlamaModel::forward(kanso_cuda_kv* kv, const StepBatch& b, float* logits
   KANSO_CUDA_TRY(ctx, cudaMemcpyAsync(d_in, p, words * 4, cudaMemcpyHostToDevice, ctx->stream),
                  "h2d");
   float* all = (float*)ctx->stage_dev;
-  st = decode_device(kv, d_in, d_in + B, d_in + 2 * B, d_in + 4 * B, d_in + 3 * B, B,
+  st = decode_device(kv, d_in, d_in + B, d_in + 2 * B, d_in + 4 * B, d_in + 3 * B, nullptr, B,
                      b.max_blocks, max_ctx, KANSO_ACT_F32, all);
   if (st) return st;
   for (uint32_t i = 0; i < b.n_want; ++i)
@@ -332,7 +333,7 @@ int32_t LlamaModel::forward(kanso_cuda_kv* kv, const StepBatch& b, float* logits
 int32_t LlamaModel::decode_device(kanso_cuda_kv* kv, const uint32_t* tokens,
                                   const uint32_t* positions, const uint32_t* slots,
                                   const uint32_t* block_tables, const uint32_t* context_lens,
-                                  uint32_t B, uint32_t max_blocks, uint32_t max_ctx,
+                                  const uint32_t*, uint32_t B, uint32_t max_blocks, uint32_t max_ctx,
                                   int32_t act_mode, float* logits_dev) {
   LlamaModel* m = this;
   const auto& c = m->cfg;

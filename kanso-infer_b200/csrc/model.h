@@ -9,7 +9,8 @@
 namespace kanso {
 
 // One ragged step, host arrays. Sequence s brings query_lens[s] tokens, the last ones of its
-// context_lens[s]; its cache pages are tables[s * max_blocks ...]. `want` names rows of the step
+// context_lens[s]; its cache pages are tables[s * max_blocks ...] and its recurrent state, where the
+// model has one, lies in slot state_slots[s] (nullptr: slot s). `want` names rows of the step
 // (0 .. T-1, ascending or not) whose logits are asked for.
 struct StepBatch {
   uint32_t S = 0, T = 0, max_blocks = 0;
@@ -17,6 +18,7 @@ struct StepBatch {
   const uint32_t* query_lens = nullptr;
   const uint32_t* context_lens = nullptr;
   const uint32_t* tables = nullptr;
+  const uint32_t* state_slots = nullptr;
   const uint32_t* want = nullptr;
   uint32_t n_want = 0;
 };
@@ -42,15 +44,18 @@ struct kanso_cuda_model {
   virtual uint32_t max_query_len() const = 0;
   // The widest window of its layers: keys further back are never read. 0: no window.
   virtual uint32_t max_window() const { return 0; }
-  // A pool of the geometry and element type its step reads.
-  virtual int32_t create_pool(uint32_t num_blocks, kanso_cuda_kv** out) = 0;
+  // A sequence has a state besides its pages: it needs a slot of the pool.
+  virtual bool has_state() const { return false; }
+  // A pool of the geometry and element type its step reads, with that many state slots.
+  virtual int32_t create_pool(uint32_t num_blocks, uint32_t num_slots, kanso_cuda_kv** out) = 0;
   virtual int32_t check_pool(const kanso_cuda_kv* kv) = 0;
   // One token per sequence, device arrays, asynchronous (kanso_cuda_decode_step_device).
+  // state_slots nullptr: sequence s has slot s.
   virtual int32_t decode_device(kanso_cuda_kv* kv, const uint32_t* tokens,
                                 const uint32_t* positions, const uint32_t* slots,
-                                const uint32_t* tables, const uint32_t* context_lens, uint32_t B,
-                                uint32_t max_blocks, uint32_t max_ctx, int32_t act_mode,
-                                float* logits_dev) = 0;
+                                const uint32_t* tables, const uint32_t* context_lens,
+                                const uint32_t* state_slots, uint32_t B, uint32_t max_blocks,
+                                uint32_t max_ctx, int32_t act_mode, float* logits_dev) = 0;
   // A ragged step on checked host arrays; asynchronous, logits [n_want, vocab] on the device.
   virtual int32_t forward(kanso_cuda_kv* kv, const kanso::StepBatch& b, float* logits_dev) = 0;
 };

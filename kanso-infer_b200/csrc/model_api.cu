@@ -1,5 +1,6 @@
 // Entry points that work on any model class: the registry and loading from a folder, the pool of
 // a model, the decode step and the ragged step with host arrays.
+#include <algorithm>
 #include <cstring>
 #include <fstream>
 #include <sstream>
@@ -100,6 +101,16 @@ int32_t check_step(kanso_cuda_model* m, const kanso_cuda_kv* kv, const StepBatch
     if (b.tokens[t] >= m->vocab_size())
       return fail(ctx, KANSO_ERR_SHAPE, "step: token id %u out of range (vocab %u)", b.tokens[t],
                   m->vocab_size());
+  if (m->has_state()) {
+    std::vector<bool> taken(kv->num_slots);
+    for (uint32_t s = 0; s < b.S; ++s) {
+      const uint32_t slot = b.state_slots ? b.state_slots[s] : s;
+      if (slot >= kv->num_slots || taken[slot])
+        return fail(ctx, KANSO_ERR_SHAPE, "step: state slot %u of sequence %u (the pool has %u)%s",
+                    slot, s, kv->num_slots, slot < kv->num_slots ? " is taken" : "");
+      taken[slot] = true;
+    }
+  }
   for (uint32_t i = 0; i < b.n_want; ++i)
     if (b.want[i] >= b.T)
       return fail(ctx, KANSO_ERR_SHAPE, "step: logits of row %u of %u", b.want[i], b.T);
@@ -161,8 +172,15 @@ int32_t kanso_cuda_model_load(kanso_cuda_ctx* ctx, const char* dir, int32_t comp
 int32_t kanso_cuda_model_create_pool(kanso_cuda_model* m, uint32_t num_blocks,
                                      kanso_cuda_kv** out) {
   if (!m) return fail(nullptr, KANSO_ERR_CONFIG, "model_create_pool: model is NULL");
+  // no more sequences than pages can be live
+  return kanso_cuda_model_create_pool_slots(m, num_blocks, std::min(num_blocks, 256u), out);
+}
+
+int32_t kanso_cuda_model_create_pool_slots(kanso_cuda_model* m, uint32_t num_blocks,
+                                           uint32_t num_slots, kanso_cuda_kv** out) {
+  if (!m) return fail(nullptr, KANSO_ERR_CONFIG, "model_create_pool: model is NULL");
   if (!out) return fail(m->ctx, KANSO_ERR_CONFIG, "model_create_pool: out is NULL");
-  return m->create_pool(num_blocks, out);
+  return m->create_pool(num_blocks, num_slots, out);
 }
 
 int32_t kanso_cuda_forward_step(kanso_cuda_ctx* ctx, kanso_cuda_model* m, kanso_cuda_kv* kv,
@@ -170,6 +188,15 @@ int32_t kanso_cuda_forward_step(kanso_cuda_ctx* ctx, kanso_cuda_model* m, kanso_
                                 const uint32_t* context_lens, const uint32_t* block_tables,
                                 uint32_t S, uint32_t max_blocks, const uint32_t* want,
                                 uint32_t n_want, float* logits_out) {
+  return kanso_cuda_forward_step_slots(ctx, m, kv, tokens, query_lens, context_lens, block_tables,
+                                       nullptr, S, max_blocks, want, n_want, logits_out);
+}
+
+int32_t kanso_cuda_forward_step_slots(kanso_cuda_ctx* ctx, kanso_cuda_model* m, kanso_cuda_kv* kv,
+                                      const uint32_t* tokens, const uint32_t* query_lens,
+                                      const uint32_t* context_lens, const uint32_t* block_tables,
+                                      const uint32_t* state_slots, uint32_t S, uint32_t max_blocks,
+                                      const uint32_t* want, uint32_t n_want, float* logits_out) {
   if (!ctx) return fail(nullptr, KANSO_ERR_CONFIG, "forward_step: ctx is NULL");
   if (!m || !kv) return fail(ctx, KANSO_ERR_SHAPE, "forward_step: model or pool is NULL");
   if (S == 0) return KANSO_OK;
@@ -184,6 +211,7 @@ int32_t kanso_cuda_forward_step(kanso_cuda_ctx* ctx, kanso_cuda_model* m, kanso_
   b.query_lens = query_lens;
   b.context_lens = context_lens;
   b.tables = block_tables;
+  b.state_slots = state_slots;
   b.want = want;
   b.n_want = n_want;
   int32_t st = run_step(m, kv, b);
@@ -202,11 +230,24 @@ int32_t kanso_cuda_decode_step_device(kanso_cuda_ctx* ctx, kanso_cuda_model* m, 
                                       const uint32_t* context_lens, uint32_t B,
                                       uint32_t max_blocks, uint32_t max_ctx, int32_t act_mode,
                                       float* logits_dev) {
+  return kanso_cuda_decode_step_device_slots(ctx, m, kv, tokens, positions, slots, block_tables,
+                                             context_lens, nullptr, B, max_blocks, max_ctx,
+                                             act_mode, logits_dev);
+}
+
+int32_t kanso_cuda_decode_step_device_slots(kanso_cuda_ctx* ctx, kanso_cuda_model* m,
+                                            kanso_cuda_kv* kv, const uint32_t* tokens,
+                                            const uint32_t* positions, const uint32_t* slots,
+                                            const uint32_t* block_tables,
+                                            const uint32_t* context_lens,
+                                            const uint32_t* state_slots, uint32_t B,
+                                            uint32_t max_blocks, uint32_t max_ctx,
+                                            int32_t act_mode, float* logits_dev) {
   if (!ctx) return fail(nullptr, KANSO_ERR_CONFIG, "decode_step: ctx is NULL");
   if (!m || !kv) return fail(ctx, KANSO_ERR_SHAPE, "decode_step: model or pool is NULL");
   if (B == 0) return KANSO_OK;
-  return m->decode_device(kv, tokens, positions, slots, block_tables, context_lens, B, max_blocks,
-                          max_ctx, act_mode, logits_dev);
+  return m->decode_device(kv, tokens, positions, slots, block_tables, context_lens, state_slots, B,
+                          max_blocks, max_ctx, act_mode, logits_dev);
 }
 
 int32_t kanso_cuda_decode_step(kanso_cuda_ctx* ctx, kanso_cuda_model* m, kanso_cuda_kv* kv,
@@ -260,7 +301,7 @@ int32_t kanso_cuda_decode_step(kanso_cuda_ctx* ctx, kanso_cuda_model* m, kanso_c
   cudaStream_t s = ctx->stream;
   KANSO_CUDA_TRY(ctx, cudaMemcpyAsync(m->d_in, ph, 4 * nb + tb, cudaMemcpyHostToDevice, s), "h2d");
   st = m->decode_device(kv, m->d_in, m->d_in + B, m->d_in + 2 * B, m->d_in + 4 * B, m->d_in + 3 * B,
-                        B, max_blocks, max_ctx, act_mode, m->logits);
+                        nullptr, B, max_blocks, max_ctx, act_mode, m->logits);
   if (st) return st;
   char* pl = ph + 4 * nb + tb;
   KANSO_CUDA_TRY(ctx, cudaMemcpyAsync(pl, m->logits, lb, cudaMemcpyDeviceToHost, s), "d2h");

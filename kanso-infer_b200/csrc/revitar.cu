@@ -17,12 +17,8 @@
 // the tile kernels, ten a layer. The residual stream, norms, scores, routing and all
 // accumulation are f32 in both number formats.
 #include <algorithm>
-#include <cstring>
-#include <memory>
 
-#include "dense.cuh"
-#include "model.h"
-#include "safetensors.h"
+#include "dense_model.h"
 
 namespace kanso {
 namespace {
@@ -37,36 +33,6 @@ struct RevConfig {
   float embed_scale = 1.f, eps = 0.f, mult = 1.f;
   std::vector<RevLayerSpec> layers;
 };
-
-// A number at a dotted path below `j`.
-int32_t need_num(kanso_cuda_ctx* ctx, const Json& j, const char* path, double* out) {
-  const Json* at = &j;
-  std::string rest(path);
-  while (at && !rest.empty()) {
-    const size_t dot = rest.find('.');
-    at = at->find(rest.substr(0, dot).c_str());
-    rest = dot == std::string::npos ? "" : rest.substr(dot + 1);
-  }
-  if (!at || at->kind != Json::NUM)
-    return fail(ctx, KANSO_ERR_CONFIG, "config.json: '%s' is missing or not a number", path);
-  *out = at->num;
-  return KANSO_OK;
-}
-int32_t need_size(kanso_cuda_ctx* ctx, const Json& j, const char* path, uint32_t* out) {
-  double v = 0;
-  const int32_t st = need_num(ctx, j, path, &v);
-  if (st) return st;
-  if (v < 1 || v > 2147483647.0 || v != (double)(uint32_t)v)
-    return fail(ctx, KANSO_ERR_CONFIG, "config.json: '%s' is not a positive whole number", path);
-  *out = (uint32_t)v;
-  return KANSO_OK;
-}
-int32_t need_float(kanso_cuda_ctx* ctx, const Json& j, const char* path, float* out) {
-  double v = 0;
-  const int32_t st = need_num(ctx, j, path, &v);
-  *out = (float)v;
-  return st;
-}
 
 int32_t parse_config(kanso_cuda_ctx* ctx, const Json& j, RevConfig* c) {
   int32_t st;
@@ -130,184 +96,39 @@ struct RevLayer {
   SigmoidAttn attn;
 };
 
-// Rows of the step on the device and what the host knows of them.
-struct RevStep {
-  int64_t T = 0;
-  const uint32_t* tokens = nullptr;
-  RowMap map;
-  const uint32_t* want = nullptr;  // nullptr: every row
-  int64_t n_want = 0;
-  const AttnTile *tiles128 = nullptr, *tiles64 = nullptr;  // the rows in tiles of that many
-  uint32_t n_tiles128 = 0, n_tiles64 = 0;
-  bool one_each = false;  // one row per sequence
-  bool use_tiles = false;
-  uint32_t max_keys = 0;
-};
-
-struct RevitarModel final : kanso_cuda_model {
+struct RevitarModel final : DenseModel {
   RevConfig cfg;
-  int32_t compute = KANSO_COMPUTE_BF16;
   std::vector<RevLayer> layers;
   DenseMat embed, head;
   float* final_norm = nullptr;
-  std::vector<void*> owned;
   // workspace of `ws_rows` rows
-  int64_t ws_rows = 0;
   int ws_parts = 1;
-  void* ws = nullptr;
   float *x = nullptr, *x2 = nullptr, *qkv = nullptr, *oy = nullptr, *ao32 = nullptr,
         *rl = nullptr, *wgt = nullptr, *act32 = nullptr, *ye = nullptr;
   void *xe = nullptr, *q = nullptr, *ao = nullptr, *xs = nullptr, *act = nullptr;
   uint32_t *sel = nullptr, *slot = nullptr, *counts = nullptr, *offsets = nullptr;
   size_t counts_bytes = 0;
-  std::vector<uint32_t> step_in;  // host image of a step's inputs
 
-  ~RevitarModel() override {
-    for (void* p : owned) cudaFree(p);
-    if (ws) cudaFree(ws);
-  }
   const char* architecture() const override { return "Revitar"; }
   uint32_t vocab_size() const override { return cfg.vocab; }
   uint32_t num_layers() const override { return (uint32_t)cfg.layers.size(); }
-  uint32_t block_size() const override { return 16; }
-  uint32_t max_positions() const override { return 0; }
-  uint32_t max_query_len() const override { return 0; }
   uint32_t max_window() const override { return widest_window(cfg); }
-  size_t elem() const { return compute == KANSO_COMPUTE_BF16 ? 2 : 4; }
-  int32_t kv_type() const {
-    return compute == KANSO_COMPUTE_BF16 ? KANSO_KV_BF16 : KANSO_KV_F32;
-  }
-  int32_t create_pool(uint32_t num_blocks, kanso_cuda_kv** out) override {
-    std::vector<uint32_t> g, k, v;
-    for (const RevLayerSpec& s : cfg.layers) {
-      g.push_back(s.kv_heads);
-      k.push_back(s.dim);
-      v.push_back(s.vdim);
-    }
-    return kanso_cuda_kv_create_dense(ctx, num_layers(), g.data(), k.data(), v.data(), num_blocks,
-                                      block_size(), kv_type(), out);
-  }
-  int32_t check_pool(const kanso_cuda_kv* kv) override {
-    bool ok = kv->kv_type == kv_type() && kv->dense.size() == cfg.layers.size();
-    for (size_t i = 0; ok && i < cfg.layers.size(); ++i) {
-      const KvDenseLayer& d = kv->dense[i];
-      const RevLayerSpec& s = cfg.layers[i];
-      ok = d.kv_heads == s.kv_heads && d.k_dim == s.dim && d.v_dim == s.vdim;
-    }
-    return ok ? KANSO_OK
-              : fail(ctx, KANSO_ERR_SHAPE, "the pool's geometry or element type is not the model's");
+  std::vector<kanso_kv_layer> cache_layers() const override {
+    std::vector<kanso_kv_layer> v;
+    for (const RevLayerSpec& s : cfg.layers) v.push_back({s.kv_heads, s.dim, s.vdim, 0, 0, 0});
+    return v;
   }
 
   int32_t load(const SafeTensors& st);
-  int32_t decode_device(kanso_cuda_kv* kv, const uint32_t* tokens, const uint32_t* positions,
-                        const uint32_t* slots, const uint32_t* tables,
-                        const uint32_t* context_lens, uint32_t B, uint32_t max_blocks,
-                        uint32_t max_ctx, int32_t act_mode, float* logits_dev) override;
-  int32_t forward(kanso_cuda_kv* kv, const StepBatch& b, float* logits_dev) override;
 
  private:
-  int32_t tensor(const SafeTensors& st, const std::string& name, std::vector<int64_t> shape,
-                 const StTensor** out);
-  int32_t upload(const void* host, size_t bytes, void** out);
-  int32_t vec(const SafeTensors& st, const std::string& name, int64_t n, float** out,
-              std::vector<float>* host = nullptr);
-  int32_t mat(const std::vector<const StTensor*>& parts, int64_t groups, int64_t cols, bool f32,
-              DenseMat* out);
   int32_t ensure_ws(int64_t T);
-  int32_t run(kanso_cuda_kv* kv, const RevStep& s, float* logits_dev);
-  int32_t run_rows(kanso_cuda_kv* kv, const RevStep& s, float* logits_dev);
-  int32_t run_tiles(kanso_cuda_kv* kv, const RevStep& s, float* logits_dev);
-  int32_t attend(kanso_cuda_kv* kv, size_t l, const RevStep& s, const QkvSource& src, void* out,
+  int32_t run(kanso_cuda_kv* kv, const DenseStep& s, float* logits_dev) override;
+  int32_t run_rows(kanso_cuda_kv* kv, const DenseStep& s, float* logits_dev);
+  int32_t run_tiles(kanso_cuda_kv* kv, const DenseStep& s, float* logits_dev);
+  int32_t attend(kanso_cuda_kv* kv, size_t l, const DenseStep& s, const QkvSource& src, void* out,
                  bool out_f32, int64_t out_ld);
 };
-
-float st_value(const StTensor& t, int64_t i) {
-  if (t.type == StType::BF16) {
-    uint16_t h;
-    std::memcpy(&h, t.data + 2 * i, 2);
-    const uint32_t u = (uint32_t)h << 16;
-    float f;
-    std::memcpy(&f, &u, 4);
-    return f;
-  }
-  float f;
-  std::memcpy(&f, t.data + 4 * i, 4);
-  return f;
-}
-uint16_t bf16_bits(float f) {  // round to nearest, ties to even
-  uint32_t u;
-  std::memcpy(&u, &f, 4);
-  if ((u & 0x7FFFFFFFu) > 0x7F800000u) return (uint16_t)((u >> 16) | 0x40u);
-  return (uint16_t)((u + 0x7FFFu + ((u >> 16) & 1u)) >> 16);
-}
-
-int32_t RevitarModel::tensor(const SafeTensors& st, const std::string& name,
-                             std::vector<int64_t> shape, const StTensor** out) {
-  const StTensor* t = st.find(name);
-  if (!t) return fail(ctx, KANSO_ERR_CONFIG, "tensor '%s' is missing", name.c_str());
-  if (t->shape != shape || t->type == StType::I32) {
-    std::string want, got;
-    for (int64_t d : shape) want += " " + std::to_string(d);
-    for (int64_t d : t->shape) got += " " + std::to_string(d);
-    return fail(ctx, KANSO_ERR_SHAPE, "tensor '%s' is [%s ], the configuration needs [%s ]",
-                name.c_str(), got.c_str(), want.c_str());
-  }
-  *out = t;
-  return KANSO_OK;
-}
-
-int32_t RevitarModel::upload(const void* host, size_t bytes, void** out) {
-  KANSO_CUDA_TRY(ctx, cudaMalloc(out, std::max<size_t>(bytes, 16)), "weights");
-  owned.push_back(*out);
-  KANSO_CUDA_TRY(ctx, cudaMemcpy(*out, host, bytes, cudaMemcpyHostToDevice), "weights");
-  return KANSO_OK;
-}
-
-int32_t RevitarModel::vec(const SafeTensors& st, const std::string& name, int64_t n, float** out,
-                          std::vector<float>* host) {
-  const StTensor* t = nullptr;
-  int32_t e = tensor(st, name, {n}, &t);
-  if (e) return e;
-  std::vector<float> v((size_t)n);
-  for (int64_t i = 0; i < n; ++i) v[(size_t)i] = st_value(*t, i);
-  if (out && (e = upload(v.data(), v.size() * 4, (void**)out))) return e;
-  if (host) *host = std::move(v);
-  return KANSO_OK;
-}
-
-// The parts' rows one under the other, `groups` equal groups of them, columns padded to 8.
-int32_t RevitarModel::mat(const std::vector<const StTensor*>& parts, int64_t groups, int64_t cols,
-                          bool f32, DenseMat* out) {
-  int64_t rows = 0;
-  for (const StTensor* t : parts) rows += t->shape[0];
-  const int64_t ld = round_up8(cols);
-  const size_t es = f32 ? 4 : 2;
-  std::vector<uint8_t> host((size_t)(rows * ld) * es, 0);
-  int64_t r = 0;
-  for (const StTensor* t : parts)
-    for (int64_t i = 0; i < t->shape[0]; ++i, ++r) {
-      uint8_t* dst = host.data() + (size_t)(r * ld) * es;
-      const int64_t at = i * cols;
-      if (f32) {
-        for (int64_t c = 0; c < cols; ++c) {
-          const float v = st_value(*t, at + c);
-          std::memcpy(dst + 4 * c, &v, 4);
-        }
-      } else if (t->type == StType::BF16) {
-        std::memcpy(dst, t->data + 2 * at, (size_t)cols * 2);
-      } else {
-        for (int64_t c = 0; c < cols; ++c) {
-          const uint16_t v = bf16_bits(st_value(*t, at + c));
-          std::memcpy(dst + 2 * c, &v, 2);
-        }
-      }
-    }
-  out->rows = rows / groups;
-  out->cols = cols;
-  out->ld = ld;
-  out->groups = groups;
-  return upload(host.data(), host.size(), &out->w);
-}
 
 int32_t RevitarModel::load(const SafeTensors& st) {
   const bool f32 = compute == KANSO_COMPUTE_F32;
@@ -363,10 +184,6 @@ int32_t RevitarModel::load(const SafeTensors& st) {
 
 int32_t RevitarModel::ensure_ws(int64_t T) {
   if (T <= ws_rows) return KANSO_OK;
-  cudaStreamSynchronize(ctx->stream);
-  if (ws) cudaFree(ws);
-  ws = nullptr;
-  ws_rows = 0;
   ws_parts = T <= 512 ? 4 : 1;
   int64_t n_qkv = 0, n_q = 0, n_o = 0, ne = 0, nt = 0, nact = 0, nact32 = 0;
   for (const RevLayerSpec& s : cfg.layers) {
@@ -381,10 +198,8 @@ int32_t RevitarModel::ensure_ws(int64_t T) {
   const int64_t W = cfg.width, WL = round_up8(W);
   const size_t es = elem();
   counts_bytes = cfg.layers.size() * (size_t)ne * 4;
-  struct {
-    void** p;
-    size_t bytes;
-  } parts[] = {{(void**)&x, (size_t)(T * W) * 4},
+  return make_ws(T,
+              {{(void**)&x, (size_t)(T * W) * 4},
                {(void**)&x2, (size_t)(T * W) * 4},
                {(void**)&qkv, (size_t)(ws_parts * T * n_qkv) * 4},
                {(void**)&oy, (size_t)(ws_parts * T * W) * 4},
@@ -401,23 +216,11 @@ int32_t RevitarModel::ensure_ws(int64_t T) {
                {(void**)&sel, (size_t)(T * nt) * 4},
                {(void**)&slot, (size_t)(T * nt) * 4},
                {(void**)&counts, counts_bytes},
-               {(void**)&offsets, (size_t)(ne + 1) * 4}};
-  size_t total = 0;
-  for (auto& b : parts) total += (b.bytes + 255) & ~(size_t)255;
-  KANSO_CUDA_TRY(ctx, cudaMalloc(&ws, std::max<size_t>(total, 256)), "workspace");
-  // pad columns are multiplied by zero: they must be finite
-  KANSO_CUDA_TRY(ctx, cudaMemsetAsync(ws, 0, total, ctx->stream), "workspace");
-  uint8_t* at = static_cast<uint8_t*>(ws);
-  for (auto& b : parts) {
-    *b.p = at;
-    at += (b.bytes + 255) & ~(size_t)255;
-  }
-  ws_rows = T;
-  return KANSO_OK;
+               {(void**)&offsets, (size_t)(ne + 1) * 4}});
 }
 
 // The attention of layer l from its projections: stores k and v and leaves the heads' outputs.
-int32_t RevitarModel::attend(kanso_cuda_kv* kv, size_t l, const RevStep& s, const QkvSource& src,
+int32_t RevitarModel::attend(kanso_cuda_kv* kv, size_t l, const DenseStep& s, const QkvSource& src,
                              void* out, bool out_f32, int64_t out_ld) {
   const RevLayer& ly = layers[l];
   const KvDenseLayer& pool = kv->dense[l];
@@ -439,7 +242,7 @@ int32_t RevitarModel::attend(kanso_cuda_kv* kv, size_t l, const RevStep& s, cons
                                   out_f32, out_ld, s.T);
 }
 
-int32_t RevitarModel::run(kanso_cuda_kv* kv, const RevStep& s, float* logits_dev) {
+int32_t RevitarModel::run(kanso_cuda_kv* kv, const DenseStep& s, float* logits_dev) {
   int32_t st = ensure_ws(s.T);
   if (st) return st;
   // the row-streaming down product keeps a row's chosen experts' activations in shared memory
@@ -452,7 +255,7 @@ int32_t RevitarModel::run(kanso_cuda_kv* kv, const RevStep& s, float* logits_dev
 // One or two rows: six launches per layer. The residual step of a sublayer runs in front of the
 // product that reads its result: the router's for the attention, the next layer's qkv for the
 // experts.
-int32_t RevitarModel::run_rows(kanso_cuda_kv* kv, const RevStep& s, float* logits_dev) {
+int32_t RevitarModel::run_rows(kanso_cuda_kv* kv, const DenseStep& s, float* logits_dev) {
   const int T = (int)s.T;
   const int64_t W = cfg.width;
   int32_t st;
@@ -471,7 +274,7 @@ int32_t RevitarModel::run_rows(kanso_cuda_kv* kv, const RevStep& s, float* logit
       ResidualSource r;
       r.y = y;
       const int32_t e = launch_residual_norm(ctx, compute, cur, W, r, y_norm, cfg.eps, cfg.mult,
-                                             nullptr, 0, T);
+                                             Residual::kAdd, nullptr, 0, T);
       if (e) return e;
       y = nullptr;
     }
@@ -505,8 +308,8 @@ int32_t RevitarModel::run_rows(kanso_cuda_kv* kv, const RevStep& s, float* logit
     if (!sp.experts) continue;
     if ((st = source(&g))) return st;
     if ((st = launch_gemv(ctx, KANSO_COMPUTE_F32, ly.router, g, rl, sp.experts, T))) return st;
-    if ((st = launch_gemv_gate_up(ctx, compute, ly.gate, ly.up, cur, rl, sp.experts, sp.top, act32,
-                                  sel, T)))
+    if ((st = launch_gemv_gate_up(ctx, compute, &ly.gate, ly.up, cur, rl, sp.experts, sp.top,
+                                  RouteWeights::kShares, act32, sel, T)))
       return st;
     if ((st = launch_gemv_down(ctx, compute, ly.down, act32, sel, sp.top, ye, T))) return st;
     y = ye;
@@ -520,7 +323,7 @@ int32_t RevitarModel::run_rows(kanso_cuda_kv* kv, const RevStep& s, float* logit
   return launch_gemv(ctx, compute, head, g, logits_dev, cfg.vocab, (int)s.n_want);
 }
 
-int32_t RevitarModel::run_tiles(kanso_cuda_kv* kv, const RevStep& s, float* logits_dev) {
+int32_t RevitarModel::run_tiles(kanso_cuda_kv* kv, const DenseStep& s, float* logits_dev) {
   const int64_t T = s.T, W = cfg.width, WL = round_up8(W);
   int32_t st;
   int splits = 1;
@@ -552,11 +355,13 @@ int32_t RevitarModel::run_tiles(kanso_cuda_kv* kv, const RevStep& s, float* logi
     r.y = oy;
     r.parts = splits;
     r.part_stride = T * W;
-    if ((st = launch_residual_norm(ctx, compute, x, W, r, ly.norm1, cfg.eps, cfg.mult, xe, WL, T)))
+    if ((st = launch_residual_norm(ctx, compute, x, W, r, ly.norm1, cfg.eps, cfg.mult,
+                                   Residual::kAdd, xe, WL, T)))
       return st;
     if (!sp.experts) continue;
     uint32_t* cnt = counts + l * count_step;
-    if ((st = launch_route(ctx, x, W, ly.router, sp.top, sel, wgt, cnt, slot, T))) return st;
+    if ((st = launch_route(ctx, x, W, ly.router, nullptr, sp.top, RouteWeights::kShares, sel, wgt,
+                           cnt, slot, T))) return st;
     if ((st = launch_expert_gather(ctx, compute, cnt, sp.experts, sp.top, sel, slot, offsets, xe,
                                    WL, xs, T)))
       return st;
@@ -571,106 +376,11 @@ int32_t RevitarModel::run_tiles(kanso_cuda_kv* kv, const RevStep& s, float* logi
     r.slot = slot;
     r.weight = wgt;
     r.top = (int)sp.top;
-    if ((st = launch_residual_norm(ctx, compute, x, W, r, ly.norm2, cfg.eps, cfg.mult, xe, WL, T)))
+    if ((st = launch_residual_norm(ctx, compute, x, W, r, ly.norm2, cfg.eps, cfg.mult,
+                                   Residual::kAdd, xe, WL, T)))
       return st;
   }
-  if (!s.n_want) return KANSO_OK;
-  if (s.n_want <= GEMV_MAX_T) {
-    GemvSource g;
-    g.x = x;
-    g.eps = cfg.eps;
-    g.final_w = final_norm;
-    g.row_index = s.want;
-    return launch_gemv(ctx, compute, head, g, logits_dev, cfg.vocab, (int)s.n_want);
-  }
-  // wanted rows in portions of the workspace (a row may be asked for more than once)
-  for (int64_t i = 0; i < s.n_want; i += T) {
-    const int64_t n = std::min(T, s.n_want - i);
-    if ((st = launch_norm_rows(ctx, compute, x, W, s.want ? s.want + i : nullptr, final_norm,
-                               cfg.eps, xe, WL, n)))
-      return st;
-    GemmRows hr;
-    hr.T = n;
-    if ((st = launch_gemm(ctx, compute, head, xe, logits_dev + i * cfg.vocab, cfg.vocab, hr, 1,
-                          &splits, 0)))
-      return st;
-  }
-  return KANSO_OK;
-}
-
-int32_t RevitarModel::decode_device(kanso_cuda_kv* kv, const uint32_t* tokens,
-                                    const uint32_t* positions, const uint32_t*,
-                                    const uint32_t* tables, const uint32_t*, uint32_t B,
-                                    uint32_t max_blocks, uint32_t max_ctx, int32_t act_mode,
-                                    float* logits_dev) {
-  if (act_mode != KANSO_ACT_F32)
-    return fail(ctx, KANSO_ERR_UNSUPPORTED, "decode_step: quantised activations need quantised "
-                                            "weights");
-  const int32_t st = check_pool(kv);
-  if (st) return st;
-  RevStep s;
-  s.T = B;
-  s.tokens = tokens;
-  s.map.positions = positions;  // a token's slot is where the table places its position
-  s.map.tables = tables;
-  s.map.max_blocks = max_blocks;
-  s.n_want = B;
-  s.one_each = true;
-  s.max_keys = max_ctx;
-  return run(kv, s, logits_dev);
-}
-
-int32_t RevitarModel::forward(kanso_cuda_kv* kv, const StepBatch& b, float* logits_dev) {
-  // the prompt kernels' tiles; short queries go row by row
-  std::vector<AttnTile> tiles, tiles64;
-  RevStep s;
-  s.T = b.T;
-  s.n_want = b.n_want;
-  s.one_each = true;
-  uint32_t row = 0;
-  const size_t words = 3 * (size_t)b.T + b.n_want + (size_t)b.S * b.max_blocks;
-  step_in.resize(words);
-  uint32_t *tok = step_in.data(), *pos = tok + b.T, *seq = pos + b.T, *want = seq + b.T,
-           *tab = want + b.n_want;
-  for (uint32_t i = 0; i < b.S; ++i) {
-    const uint32_t n = b.query_lens[i], c = b.context_lens[i], p0 = c - n;
-    s.one_each = s.one_each && n == 1;
-    s.use_tiles = s.use_tiles || n >= 16;
-    s.max_keys = std::max(s.max_keys, c);
-    for (uint32_t k = 0; k < n; k += 128)
-      tiles.push_back({row + k, std::min(128u, n - k), p0 + k, i});
-    for (uint32_t k = 0; k < n; k += 64)
-      tiles64.push_back({row + k, std::min(64u, n - k), p0 + k, i});
-    for (uint32_t k = 0; k < n; ++k, ++row) {
-      pos[row] = p0 + k;
-      seq[row] = i;
-    }
-  }
-  std::memcpy(tok, b.tokens, (size_t)b.T * 4);
-  if (b.n_want) std::memcpy(want, b.want, (size_t)b.n_want * 4);
-  std::memcpy(tab, b.tables, (size_t)b.S * b.max_blocks * 4);
-  static_assert(sizeof(AttnTile) == 16, "four words");
-  s.n_tiles128 = (uint32_t)tiles.size();
-  s.n_tiles64 = (uint32_t)tiles64.size();
-  tiles.insert(tiles.end(), tiles64.begin(), tiles64.end());
-  const size_t tile_at = (words + 3) & ~(size_t)3;
-  step_in.resize(tile_at + 4 * tiles.size());
-  std::memcpy(step_in.data() + tile_at, tiles.data(), tiles.size() * sizeof(AttnTile));
-  int32_t st = model_inputs(this, step_in.size());
-  if (st) return st;
-  KANSO_CUDA_TRY(ctx,
-                 cudaMemcpyAsync(d_in, step_in.data(), step_in.size() * 4, cudaMemcpyHostToDevice,
-                                 ctx->stream),
-                 "h2d");
-  s.tokens = d_in;
-  s.map.positions = d_in + b.T;
-  s.map.row_seq = d_in + 2 * (size_t)b.T;
-  s.want = d_in + 3 * (size_t)b.T;
-  s.map.tables = s.want + b.n_want;
-  s.map.max_blocks = b.max_blocks;
-  s.tiles128 = reinterpret_cast<const AttnTile*>(d_in + tile_at);
-  s.tiles64 = s.tiles128 + s.n_tiles128;
-  return run(kv, s, logits_dev);
+  return logits_of_rows(head, final_norm, cfg.eps, x, xe, s, logits_dev);
 }
 
 int32_t describe(kanso_cuda_ctx* ctx, const Json& config, std::string* summary) {

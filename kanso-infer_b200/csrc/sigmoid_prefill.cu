@@ -19,6 +19,7 @@
 #include "dense.cuh"
 #include "tc05.cuh"
 #include "tensor_map.h"
+#include "warp_mma.cuh"
 
 namespace kanso {
 
@@ -41,51 +42,6 @@ struct PrefillArgs {
   uint32_t tmem_cols;
   int* status;
 };
-
-__device__ __forceinline__ void sp_tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,"
-      "%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]),
-        "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]),
-        "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]),
-        "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]),
-        "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-      : "r"(taddr)
-      : "memory");
-  asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-}
-__device__ __forceinline__ float sp_ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ float sp_rcp(float x) {
-  float y;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-// Bounded, and ends early when another role has given up.
-__device__ __forceinline__ bool sp_wait(uint64_t* bar, uint32_t parity, volatile int* abort_flag) {
-  for (uint32_t i = 0; i < (1u << 22); ++i) {
-    if (mbar_try_wait(bar, parity)) return true;
-    if ((i & 63u) == 63u && *abort_flag) break;
-  }
-  *abort_flag = 1;
-  return false;
-}
-
-// N-major operand in the 128-byte swizzle: panels of 64 columns, `panel` bytes apart, of rows of
-// 128 bytes (one per k), groups of eight rows 1024 bytes apart. 16 k further is 2048 bytes.
-__device__ __forceinline__ uint64_t sp_desc_nmajor(uint32_t addr, uint32_t panel) {
-  uint64_t d = 0;
-  d |= (uint64_t)((addr >> 4) & 0x3FFF);
-  d |= (uint64_t)((panel >> 4) & 0x3FFF) << 16;
-  d |= (uint64_t)(1024 >> 4) << 32;
-  d |= (uint64_t)1 << 46;
-  d |= (uint64_t)2 << 61;
-  return d;
-}
 
 __global__ void __launch_bounds__(SP_THREADS, 1)
     sigmoid_prefill_kernel(const __grid_constant__ CUtensorMap qmap,
@@ -174,7 +130,7 @@ __global__ void __launch_bounds__(SP_THREADS, 1)
       const int s = i % SP_STAGES;
       const uint32_t par = ((uint32_t)(i / SP_STAGES) & 1u) ^ 1u;
       const uint32_t next = i + 1 < n_tiles ? page_of(i + 1) : 0u;
-      bool ok = sp_wait(&k_empty[s], par, &abort_flag);
+      bool ok = mbar_wait_abort(&k_empty[s], par, &abort_flag);
       if (lane == 0 && ok) mbar_arrive_expect_tx(&k_full[s], k_bytes);
       __syncwarp();
       ok = __all_sync(0xFFFFFFFFu, ok);
@@ -185,7 +141,7 @@ __global__ void __launch_bounds__(SP_THREADS, 1)
           tma_load_3d(Ks + (size_t)s * k_bytes + (size_t)c * SP_K * 128 +
                           (size_t)lane * p.block_size * 128,
                       &kmap, c * 64, 0, rec, &k_full[s]);
-      ok = sp_wait(&v_empty[s], par, &abort_flag);
+      ok = mbar_wait_abort(&v_empty[s], par, &abort_flag);
       if (lane == 0 && ok) mbar_arrive_expect_tx(&v_full[s], v_bytes);
       __syncwarp();
       ok = __all_sync(0xFFFFFFFFu, ok);
@@ -212,10 +168,10 @@ __global__ void __launch_bounds__(SP_THREADS, 1)
     if (lane == 0) {
       const uint32_t id_s = tc_idesc_bf16(SP_Q, SP_K);
       const uint32_t id_o = tc_idesc_bf16(SP_Q, p.nv) | (1u << 16);  // B is N-major
-      bool ok = sp_wait(&q_full, 0, &abort_flag);
+      bool ok = mbar_wait_abort(&q_full, 0, &abort_flag);
       auto scores = [&](int i) {
         const int s = i % SP_STAGES;
-        if (ok) ok = sp_wait(&k_full[s], (uint32_t)(i / SP_STAGES) & 1u, &abort_flag);
+        if (ok) ok = mbar_wait_abort(&k_full[s], (uint32_t)(i / SP_STAGES) & 1u, &abort_flag);
         if (!ok) return;
         tc_fence_after();
         for (int k = 0; k < p.k_steps; ++k) {
@@ -234,18 +190,18 @@ __global__ void __launch_bounds__(SP_THREADS, 1)
         const int b = i & 1, s = i % SP_STAGES;
         const uint32_t par = (uint32_t)(i >> 1) & 1u;
         if (i + 2 < n_tiles) {
-          ok = sp_wait(&s_free[b], par, &abort_flag);
+          ok = mbar_wait_abort(&s_free[b], par, &abort_flag);
           if (!ok) break;
           tc_fence_after();
           scores(i + 2);
         }
-        if (ok) ok = sp_wait(&v_full[s], (uint32_t)(i / SP_STAGES) & 1u, &abort_flag);
-        if (ok) ok = sp_wait(&p_full[b], par, &abort_flag);
+        if (ok) ok = mbar_wait_abort(&v_full[s], (uint32_t)(i / SP_STAGES) & 1u, &abort_flag);
+        if (ok) ok = mbar_wait_abort(&p_full[b], par, &abort_flag);
         if (!ok) break;
         tc_fence_after();
         const uint64_t ad = tc_smem_desc_sw128(smem_u32(Ps) + (uint32_t)b * SP_P_BYTES);
         const uint64_t bd =
-            sp_desc_nmajor(smem_u32(Vs) + (uint32_t)s * v_bytes, SP_K * 128u);
+            tc_smem_desc_nmajor(smem_u32(Vs) + (uint32_t)s * v_bytes, SP_K * 128u);
 #pragma unroll
         for (int k = 0; k < SP_K / 16; ++k)
           tc_mma_f16(o_tmem, ad + 2 * k, bd + 128 * k, id_o, (i > 0 || k > 0) ? 1u : 0u);
@@ -267,8 +223,8 @@ __global__ void __launch_bounds__(SP_THREADS, 1)
     const float c1 = 2.f * cap * L2E, k0s = -L2E * p.a.scale;
     for (int i = wg; i < n_tiles; i += 2) {
       const uint32_t par = (uint32_t)(i >> 1) & 1u;
-      if (!sp_wait(&s_full[wg], par, &abort_flag)) break;
-      if (!sp_wait(&p_free[wg], par ^ 1u, &abort_flag)) break;
+      if (!mbar_wait_abort(&s_full[wg], par, &abort_flag)) break;
+      if (!mbar_wait_abort(&p_free[wg], par ^ 1u, &abort_flag)) break;
       __syncwarp();
       tc_fence_after();
       // tab index of the tile's first key; it falls by one per key
@@ -277,7 +233,7 @@ __global__ void __launch_bounds__(SP_THREADS, 1)
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         uint32_t r[32];
-        sp_tmem_ld32(s_lane + half * 32, r);
+        tmem_ld32(s_lane + half * 32, r);
         if (half == 1) {
           tc_fence_before();
           mbar_arrive(&s_free[wg]);
@@ -292,9 +248,9 @@ __global__ void __launch_bounds__(SP_THREADS, 1)
             for (int u = 0; u < 2; ++u) {
               const int col = c * 8 + e * 2 + u;
               const float s = __uint_as_float(r[col]), b = tb[-(half * 32 + col)];
-              const float arg = cap != 0.f ? fmaf(sp_rcp(1.f + sp_ex2(s * k1)), c1, b)
+              const float arg = cap != 0.f ? fmaf(rcp_approx(1.f + ex2_approx(s * k1)), c1, b)
                                            : fmaf(s, k0s, b);
-              v[u] = sp_rcp(1.f + sp_ex2(arg));
+              v[u] = rcp_approx(1.f + ex2_approx(arg));
             }
             const __nv_bfloat162 pk = __floats2bfloat162_rn(v[0], v[1]);
             w[e] = *reinterpret_cast<const uint32_t*>(&pk);
@@ -353,20 +309,6 @@ __global__ void __launch_bounds__(SP_THREADS, 1)
   if (warp == 9) tmem_dealloc(tmem, p.tmem_cols);
 }
 
-// A 3-D map of bfloat16 rows: `cols` of `mid` rows, `stride1` elements apart, of `outer` records,
-// `stride2` elements apart, read in boxes of 64 columns x box1 x box2.
-static bool map3(TmEncodeFn encode, const void* base, uint64_t cols, uint64_t mid, uint64_t outer,
-                 uint64_t stride1, uint64_t stride2, uint32_t box1, uint32_t box2,
-                 CUtensorMap* map) {
-  const cuuint64_t dim[3] = {cols, mid, outer};
-  const cuuint64_t stride[2] = {stride1 * 2, stride2 * 2};
-  const cuuint32_t box[3] = {64, box1, box2}, es[3] = {1, 1, 1};
-  return encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dim, stride, box,
-                es, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
-                CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
 int32_t launch_sigmoid_attn_prefill(kanso_cuda_ctx* ctx, const SigmoidAttn& a,
                                     const KvDenseLayer& kv, const void* q, int64_t q_rows,
                                     const RowMap& map, const AttnTile* tiles, uint32_t n_tiles,
@@ -404,10 +346,10 @@ int32_t launch_sigmoid_attn_prefill(kanso_cuda_ctx* ctx, const SigmoidAttn& a,
   const uint64_t records = (uint64_t)kv.num_blocks * kv.kv_heads;
   CUtensorMap qm, km, vm;
   const bf16* pool = reinterpret_cast<const bf16*>(kv.base);
-  if (!map3(encode, q, kv.k_ld, a.heads, (uint64_t)q_rows, kv.k_ld, (uint64_t)a.heads * kv.k_ld, 1,
+  if (!tm_map3(encode, q, kv.k_ld, a.heads, (uint64_t)q_rows, kv.k_ld, (uint64_t)a.heads * kv.k_ld, 1,
             SP_Q, &qm) ||
-      !map3(encode, pool, kv.k_ld, bs, records, kv.k_ld, kv.rec_elems, bs, 1, &km) ||
-      !map3(encode, pool + (size_t)bs * kv.k_ld, kv.v_ld, bs, records, kv.v_ld, kv.rec_elems, bs, 1,
+      !tm_map3(encode, pool, kv.k_ld, bs, records, kv.k_ld, kv.rec_elems, bs, 1, &km) ||
+      !tm_map3(encode, pool + (size_t)bs * kv.k_ld, kv.v_ld, bs, records, kv.v_ld, kv.rec_elems, bs, 1,
             &vm))
     return KANSO_OK;
   int32_t st = allow_max_smem(ctx, (const void*)sigmoid_prefill_kernel);
