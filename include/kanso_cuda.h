@@ -584,6 +584,76 @@ int32_t kanso_cuda_moe(kanso_cuda_ctx* ctx, int32_t compute, const float* x, con
                        const void* gate, const void* up, const void* down, float* y, int64_t T,
                        int64_t width, int64_t ff, uint32_t experts, uint32_t top, int32_t path);
 
+/* y = x W^T + bias (bias f32[rows] or NULL), with relu2 max(0, .)^2 of it; arguments as above. */
+int32_t kanso_cuda_dense_linear_act(kanso_cuda_ctx* ctx, int32_t compute, const void* w,
+                                    const void* x, const float* bias, int32_t relu2, float* y,
+                                    int64_t T, int64_t rows, int64_t cols, int32_t path);
+/* Routed experts without a gate: z = router_w x + router_bias (NULL: 0), the top largest chosen,
+ * weighted by the softmax over the chosen ones alone, y = sum_e s_e W_down,e max(0, W_up,e x)^2. */
+int32_t kanso_cuda_moe_relu2(kanso_cuda_ctx* ctx, int32_t compute, const float* x,
+                             const float* router, const float* router_bias, const void* up,
+                             const void* down, float* y, int64_t T, int64_t width, int64_t ff,
+                             uint32_t experts, uint32_t top, int32_t path);
+/* The residual step in place on x f32[T][width] with a sublayer's output y. after_sum 0: x += mult *
+ * rmsnorm(y) * w; 1: x = rmsnorm(mult * x + y) * w. */
+int32_t kanso_cuda_residual_norm(kanso_cuda_ctx* ctx, float* x, const float* y, const float* w,
+                                 float eps, float mult, int32_t after_sum, int64_t T,
+                                 int64_t width);
+
+/* Latent attention. A layer of the pool has one head, k_dim = rank + rot and no values; a token's
+ * row is [normed latent c | rotated key part]. Rotation turns the pairs (2i, 2i + 1) by position *
+ * rot_base^(-2i / rot). sink: HOST f32[num_heads], one more term exp(sink) of the softmax's
+ * denominator. */
+typedef struct kanso_latent_attention_params {
+  uint32_t num_rows, num_heads, max_num_blocks_per_seq;
+  uint32_t dim, rot, vdim, rank;
+  float scale;
+  double rot_base;
+  const float* sink;
+} kanso_latent_attention_params;
+/* The cache rows from the down projections f32[T][q_rank + rank + rot], and the normed query
+ * latents cq [T][q_rank rounded up to 8] in the products' element type. */
+int32_t kanso_cuda_latent_store(kanso_cuda_ctx* ctx, kanso_cuda_kv* kv, uint32_t layer,
+                                const float* down, uint32_t q_rank, const float* q_norm,
+                                const float* c_norm, float eps, const uint32_t* positions,
+                                const uint32_t* row_seq, const uint32_t* block_tables,
+                                const kanso_latent_attention_params* p, void* cq);
+/* out f32[T][num_heads][rank] = sum_j softmax_j(scale * (q_lat . c_j + q_rot . k_rot_j)) c_j over the
+ * keys at the row's position and before it. q_lat f32[T][num_heads][rank]; q f32[T][num_heads][dim +
+ * rot], of which the last rot columns are rotated and used. path: 0 = the library's choice, 1 =
+ * plain, 2 = mma.sync tiles (bfloat16; KANSO_ERR_UNSUPPORTED when a size is outside its range). */
+int32_t kanso_cuda_latent_attention(kanso_cuda_ctx* ctx, const kanso_cuda_kv* kv, uint32_t layer,
+                                    const float* q_lat, const float* q, const uint32_t* positions,
+                                    const uint32_t* row_seq, const uint32_t* block_tables,
+                                    float* out, const kanso_latent_attention_params* p,
+                                    int32_t path);
+/* Causal softmax attention of one sequence's rows pos0 .. pos0 + num_rows - 1 over its first pos0 +
+ * num_rows keys on tcgen05, all bfloat16: q [T][num_heads][dim ld], q_rot [T][num_heads][rot ld]
+ * (rotated), k [keys][num_heads][dim ld], v [keys][num_heads][vdim ld], k_rot [keys][rot ld] shared by
+ * the heads (rot 0: none), out [T][num_heads * vdim]; ld = rounded up to 8 with a zero pad. sink as
+ * above (NULL: none). KANSO_ERR_UNSUPPORTED when a size is outside the kernel's range. */
+int32_t kanso_cuda_softmax_prefill(kanso_cuda_ctx* ctx, const void* q, const void* q_rot,
+                                   const void* k, const void* v, const void* k_rot, void* out,
+                                   uint32_t pos0, const kanso_latent_attention_params* p);
+
+/* Matrix memory with exponential gates (csrc/mlstm.cu) on num_rows tokens of one sequence from
+ * position pos0, whose state lies in `slot` of the pool's layer. y f32[T][heads * (2 dim + 2 vdim +
+ * 2)] = [q | k | v | gate | i | f] as projected; i_bias, f_bias f32[heads]; out f32[T][heads * vdim].
+ * path: 0 = the library's choice, 1 = token by token, 2 = chunks on the tensor cores (bfloat16 q, k,
+ * v). */
+typedef struct kanso_mlstm_params {
+  uint32_t num_rows, pos0, slot;
+  float gate_cap;
+} kanso_mlstm_params;
+int32_t kanso_cuda_mlstm(kanso_cuda_ctx* ctx, kanso_cuda_kv* kv, uint32_t layer, const float* y,
+                         const float* i_bias, const float* f_bias, float* out,
+                         const kanso_mlstm_params* p, int32_t path);
+/* out f32[T][heads * vdim] = o with each head over its own root mean square, times w, times the
+ * sigmoid of the gate columns of y. */
+int32_t kanso_cuda_head_norm_gate(kanso_cuda_ctx* ctx, const float* o, const float* y,
+                                  const float* w, float eps, float* out, int64_t T, uint32_t heads,
+                                  uint32_t dim, uint32_t vdim);
+
 #ifdef __cplusplus
 }
 #endif

@@ -52,6 +52,19 @@ class SigmoidAttentionParams(C.Structure):
                 ("r1", C.c_void_p), ("r2", C.c_void_p), ("pb", C.c_void_p)]
 
 
+class LatentAttentionParams(C.Structure):
+    """sink is a host float32 array of num_heads (numpy), or None."""
+    _fields_ = [("num_rows", C.c_uint32), ("num_heads", C.c_uint32),
+                ("max_num_blocks_per_seq", C.c_uint32), ("dim", C.c_uint32), ("rot", C.c_uint32),
+                ("vdim", C.c_uint32), ("rank", C.c_uint32), ("scale", C.c_float),
+                ("rot_base", C.c_double), ("sink", C.c_void_p)]
+
+
+class MlstmParams(C.Structure):
+    _fields_ = [("num_rows", C.c_uint32), ("pos0", C.c_uint32), ("slot", C.c_uint32),
+                ("gate_cap", C.c_float)]
+
+
 class ModelConfig(C.Structure):
     _fields_ = [("hidden_size", C.c_uint32), ("num_attention_heads", C.c_uint32),
                 ("num_key_value_heads", C.c_uint32), ("num_hidden_layers", C.c_uint32),
@@ -152,6 +165,18 @@ PROTOTYPES = {
     "kanso_cuda_qk_norm_store": (_I32, [_P, _P, _U32, _P, _P, _P, _F, _U32, _P, _P, _P, _U32, _U32,
                                         _P]),
     "kanso_cuda_dense_linear": (_I32, [_P, _I32, _P, _P, _P, _I64, _I64, _I64, _I32]),
+    "kanso_cuda_dense_linear_act": (_I32, [_P, _I32, _P, _P, _P, _I32, _P, _I64, _I64, _I64, _I32]),
+    "kanso_cuda_moe_relu2": (_I32, [_P, _I32, _P, _P, _P, _P, _P, _P, _I64, _I64, _I64, _U32, _U32,
+                                    _I32]),
+    "kanso_cuda_residual_norm": (_I32, [_P, _P, _P, _P, _F, _F, _I32, _I64, _I64]),
+    "kanso_cuda_latent_store": (_I32, [_P, _P, _U32, _P, _U32, _P, _P, _F, _P, _P, _P,
+                                       C.POINTER(LatentAttentionParams), _P]),
+    "kanso_cuda_latent_attention": (_I32, [_P, _P, _U32, _P, _P, _P, _P, _P, _P,
+                                           C.POINTER(LatentAttentionParams), _I32]),
+    "kanso_cuda_softmax_prefill": (_I32, [_P, _P, _P, _P, _P, _P, _P, _U32,
+                                          C.POINTER(LatentAttentionParams)]),
+    "kanso_cuda_mlstm": (_I32, [_P, _P, _U32, _P, _P, _P, _P, C.POINTER(MlstmParams), _I32]),
+    "kanso_cuda_head_norm_gate": (_I32, [_P, _P, _P, _P, _F, _P, _I64, _U32, _U32, _U32]),
     "kanso_cuda_moe": (_I32, [_P, _I32, _P, _P, _P, _P, _P, _P, _I64, _I64, _I64, _U32, _U32,
                               _I32]),
 }

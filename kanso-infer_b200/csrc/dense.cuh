@@ -428,7 +428,7 @@ int32_t launch_latent_attn_rows(kanso_cuda_ctx* ctx, int32_t compute, const Late
                                 const KvDenseLayer& kv, const LatentRows& r, int path,
                                 bool* handled);
 // Causal softmax attention of prompts on tcgen05, bfloat16, over keys and values that lie one
-// after the other: k [n][heads][dim ld] with rows of kv_ld elements, v likewise, k_rot [n][rot ld]
+// after the other: k [n][heads][dim ld] with rows of k_ld elements, v likewise, k_rot [n][rot ld]
 // shared by the heads (rot 0: none); q and q_rot as launch_latent_q_rows leaves them. A tile's last
 // word is where its sequence's keys begin. sink may be nullptr. *handled = false when a size is
 // outside the kernel's range.
@@ -439,7 +439,7 @@ struct SoftmaxPrefill {
   const bf16 *q = nullptr, *q_rot = nullptr;
   int64_t q_rows = 0;
   const bf16 *k = nullptr, *v = nullptr, *k_rot = nullptr;
-  int64_t kv_ld = 0, keys = 0;
+  int64_t k_ld = 0, v_ld = 0, keys = 0;
   const AttnTile* tiles = nullptr;
   uint32_t n_tiles = 0;
   bf16* out = nullptr;  // [rows][heads * vdim], rows of out_ld

@@ -20,6 +20,11 @@ __global__ void narrow_kernel(const float* x, E* y, int64_t T, int64_t ld, int64
 }
 }  // namespace
 
+static int32_t run_moe(kanso_cuda_ctx* ctx, int32_t compute, const float* x, const float* router,
+                       const float* bias, RouteWeights form, const void* gate, const void* up,
+                       const void* down, float* y, int64_t T, int64_t width, int64_t ff,
+                       uint32_t experts, uint32_t top, int32_t path);
+
 extern "C" {
 
 int32_t kanso_cuda_sigmoid_attention(kanso_cuda_ctx* ctx, const kanso_cuda_kv* kv, uint32_t layer,
@@ -122,6 +127,12 @@ int32_t kanso_cuda_qk_norm_store(kanso_cuda_ctx* ctx, kanso_cuda_kv* kv, uint32_
 int32_t kanso_cuda_dense_linear(kanso_cuda_ctx* ctx, int32_t compute, const void* w,
                                 const void* x, float* y, int64_t T, int64_t rows, int64_t cols,
                                 int32_t path) {
+  return kanso_cuda_dense_linear_act(ctx, compute, w, x, nullptr, 0, y, T, rows, cols, path);
+}
+
+int32_t kanso_cuda_dense_linear_act(kanso_cuda_ctx* ctx, int32_t compute, const void* w,
+                                    const void* x, const float* bias, int32_t relu2, float* y,
+                                    int64_t T, int64_t rows, int64_t cols, int32_t path) {
   if (!ctx) return fail(nullptr, KANSO_ERR_CONFIG, "dense_linear: ctx is NULL");
   if (!w || !x || !y || T < 0 || rows < 1 || cols < 1)
     return fail(ctx, KANSO_ERR_SHAPE, "dense_linear: bad argument");
@@ -147,23 +158,49 @@ int32_t kanso_cuda_dense_linear(kanso_cuda_ctx* ctx, int32_t compute, const void
         return fail(ctx, KANSO_ERR_UNSUPPORTED, "dense_linear: row streaming of padded f32 rows");
       g.x = (const float*)x;
     }
-    return launch_gemv(ctx, compute, m, g, y, rows, (int)T);
+    GemvOut o;
+    o.bias = bias;
+    o.relu2 = relu2 != 0;
+    return launch_gemv(ctx, compute, m, g, y, rows, (int)T, o);
   }
   GemmRows r;
   r.T = T;
+  GemmOut o;
+  o.bias = bias;
+  o.relu2 = relu2 != 0;
   int splits = 1;
-  return launch_gemm(ctx, compute, m, x, y, rows, r, 1, &splits, 0);
+  return launch_gemm(ctx, compute, m, x, y, rows, r, 1, &splits, 0, o);
 }
 
 int32_t kanso_cuda_moe(kanso_cuda_ctx* ctx, int32_t compute, const float* x, const float* router,
                        const void* gate, const void* up, const void* down, float* y, int64_t T,
                        int64_t width, int64_t ff, uint32_t experts, uint32_t top, int32_t path) {
   if (!ctx) return fail(nullptr, KANSO_ERR_CONFIG, "moe: ctx is NULL");
-  if (!x || !router || !gate || !up || !down || !y || T < 0 || width < 1 || ff < 1 || !experts ||
-      !top || top > experts)
+  if (!gate || !aligned16(gate)) return fail(ctx, KANSO_ERR_SHAPE, "moe: bad argument");
+  return run_moe(ctx, compute, x, router, nullptr, RouteWeights::kShares, gate, up, down, y, T,
+                 width, ff, experts, top, path);
+}
+
+int32_t kanso_cuda_moe_relu2(kanso_cuda_ctx* ctx, int32_t compute, const float* x,
+                             const float* router, const float* router_bias, const void* up,
+                             const void* down, float* y, int64_t T, int64_t width, int64_t ff,
+                             uint32_t experts, uint32_t top, int32_t path) {
+  if (!ctx) return fail(nullptr, KANSO_ERR_CONFIG, "moe: ctx is NULL");
+  return run_moe(ctx, compute, x, router, router_bias, RouteWeights::kChosenSoftmax, nullptr, up,
+                 down, y, T, width, ff, experts, top, path);
+}
+
+}  // extern "C"
+
+// gate nullptr: experts of max(0, up x)^2
+static int32_t run_moe(kanso_cuda_ctx* ctx, int32_t compute, const float* x, const float* router,
+                       const float* bias, RouteWeights form, const void* gate, const void* up,
+                       const void* down, float* y, int64_t T, int64_t width, int64_t ff,
+                       uint32_t experts, uint32_t top, int32_t path) {
+  if (!x || !router || !up || !down || !y || T < 0 || width < 1 || ff < 1 || !experts || !top ||
+      top > experts)
     return fail(ctx, KANSO_ERR_SHAPE, "moe: bad argument");
-  if (!aligned16(x) || !aligned16(router) || !aligned16(gate) || !aligned16(up) ||
-      !aligned16(down) || !aligned16(y))
+  if (!aligned16(x) || !aligned16(router) || !aligned16(up) || !aligned16(down) || !aligned16(y))
     return fail(ctx, KANSO_ERR_SHAPE, "moe: arrays must be 16-byte aligned");
   if (T == 0) return KANSO_OK;
   auto mat = [&](const void* w, int64_t rows, int64_t cols, int64_t groups) {
@@ -203,9 +240,12 @@ int32_t kanso_cuda_moe(kanso_cuda_ctx* ctx, int32_t compute, const float* x, con
   if (path == 1 || (path == 0 && T <= GEMV_MAX_T)) {
     GemvSource src;
     src.x = x;
-    st = launch_gemv(ctx, KANSO_COMPUTE_F32, r, src, rl, experts, (int)T);
-    if (!st) st = launch_gemv_gate_up(ctx, compute, &g, u, x, rl, experts, top, RouteWeights::kShares,
-                                        a32, sel, (int)T);
+    GemvOut o;
+    o.bias = bias;
+    st = launch_gemv(ctx, KANSO_COMPUTE_F32, r, src, rl, experts, (int)T, o);
+    if (!st)
+      st = launch_gemv_gate_up(ctx, compute, gate ? &g : nullptr, u, x, rl, experts, top, form, a32,
+                               sel, (int)T);
     if (!st) st = launch_gemv_down(ctx, compute, d, a32, sel, top, y, (int)T);
   } else {
     if (compute == KANSO_COMPUTE_BF16)
@@ -213,8 +253,7 @@ int32_t kanso_cuda_moe(kanso_cuda_ctx* ctx, int32_t compute, const float* x, con
     else
       narrow_kernel<float><<<256, 256, 0, ctx->stream>>>(x, (float*)(mem + o_xe), T, WL, width);
     st = after_launch(ctx, "narrow");
-    if (!st) st = launch_route(ctx, x, width, r, nullptr, top, RouteWeights::kShares, sel, wgt,
-                              cnt, slot, T);
+    if (!st) st = launch_route(ctx, x, width, r, bias, top, form, sel, wgt, cnt, slot, T);
     if (!st)
       st = launch_expert_gather(ctx, compute, cnt, experts, top, sel, slot, off, mem + o_xe, WL,
                                 mem + o_xs, T);
@@ -223,7 +262,11 @@ int32_t kanso_cuda_moe(kanso_cuda_ctx* ctx, int32_t compute, const float* x, con
     er.offsets = off;
     er.groups = (int)experts;
     int splits = 1;
-    if (!st) st = launch_gemm_gate_up(ctx, compute, g, u, mem + o_xs, mem + o_act, FL, er);
+    GemmOut act;
+    act.elem = act.relu2 = true;
+    if (!st)
+      st = gate ? launch_gemm_gate_up(ctx, compute, g, u, mem + o_xs, mem + o_act, FL, er)
+                : launch_gemm(ctx, compute, u, mem + o_xs, mem + o_act, FL, er, 1, &splits, 0, act);
     if (!st) st = launch_gemm(ctx, compute, d, mem + o_act, ye, width, er, 1, &splits, 0);
     if (!st) st = launch_expert_sum(ctx, ye, slot, wgt, top, y, width, T);
   }
@@ -231,5 +274,3 @@ int32_t kanso_cuda_moe(kanso_cuda_ctx* ctx, int32_t compute, const float* x, con
   cudaFree(mem);
   return st;
 }
-
-}  // extern "C"

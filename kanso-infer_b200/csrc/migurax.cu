@@ -613,7 +613,7 @@ int32_t MiguraxModel::latent_long(kanso_cuda_kv* kv, size_t l, const DenseStep& 
   p->k = kvx;
   p->v = kvx + (int64_t)sp.heads * round_up8(sp.dim);
   p->k_rot = rot;
-  p->kv_ld = N;
+  p->k_ld = p->v_ld = N;
   p->tiles = s.long_tiles;
   p->n_tiles = s.n_long_tiles;
   p->out = (bf16*)ao;

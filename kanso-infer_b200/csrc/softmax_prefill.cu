@@ -337,8 +337,8 @@ int32_t launch_softmax_prefill(kanso_cuda_ctx* ctx, const SoftmaxPrefill& p, boo
   const uint64_t dl = round_up8(p.dim), vl = round_up8(p.vdim), rl = round_up8(p.rot), H = p.heads;
   CUtensorMap qm, qrm, km, krm, vm;
   bool ok = tm_map3(encode, p.q, dl, H, (uint64_t)p.q_rows, dl, H * dl, 1, SX_Q, &qm) &&
-            tm_map3(encode, p.k, dl, H, (uint64_t)p.keys, dl, (uint64_t)p.kv_ld, 1, SX_K, &km) &&
-            tm_map3(encode, p.v, vl, H, (uint64_t)p.keys, vl, (uint64_t)p.kv_ld, 1, SX_K, &vm);
+            tm_map3(encode, p.k, dl, H, (uint64_t)p.keys, dl, (uint64_t)p.k_ld, 1, SX_K, &km) &&
+            tm_map3(encode, p.v, vl, H, (uint64_t)p.keys, vl, (uint64_t)p.v_ld, 1, SX_K, &vm);
   qrm = qm;
   krm = km;
   if (ok && p.rot)

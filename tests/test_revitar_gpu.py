@@ -292,9 +292,12 @@ class WithMargin(np.ndarray):
 
 
 class Case:
+    """A small model on the device beside the plain statement of its class."""
+    models, weights, plain_class = MODELS, staticmethod(weights), plain
+
     def __init__(self, kb, ctx, folder, name, compute, seed=1):
-        self.cfg = MODELS[name]
-        self.w = weights(self.cfg, seed)
+        self.cfg = self.models[name]
+        self.w = self.weights(self.cfg, seed)
         self.kb, self.V, self.compute = kb, self.cfg["vocab"], compute
         self.folder = write_model(folder, self.cfg, self.w)
         self.model = kb.Model.from_dir(ctx, self.folder, compute)
@@ -304,8 +307,9 @@ class Case:
         return [int(t) for t in self.rng.integers(0, self.V, n)]
 
     def plain(self, tokens):
-        ref = plain.logits(self.cfg, self.w, tokens).view(WithMargin)
-        ref.margin = plain.routing_margin(self.cfg, self.w, tokens) if self.compute == BF16 else None
+        p = self.plain_class
+        ref = p.logits(self.cfg, self.w, tokens).view(WithMargin)
+        ref.margin = p.routing_margin(self.cfg, self.w, tokens) if self.compute == BF16 else None
         return ref
 
     def close(self, got, ref, margin=None):
