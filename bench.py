@@ -602,29 +602,10 @@ REVITAR_SIZES = {"1k": (1024, 16, 4, 64, 1024, 16, 2, 1024, 12),
 REVITAR_VOCAB = 32768
 
 
-def _write_revitar(torch, folder, size, layers=None):
-    """A Revitar model folder of that size with random bfloat16 weights; its parameter counts
-    [attention, router, one expert] per layer."""
-    W, H, G, D, window, E, top, ff, L = REVITAR_SIZES[size]
-    L = layers or L
-    one = {"type": "attention",
-           "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5,
-                     "softcap": 30.0, "mask": {"size": window}},
-           "mlp": {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": E, "top": top}}}
+def _write_model(torch, folder, config, shapes, value):
+    """A model folder with random bfloat16 weights: value(name, standard normal tensor, shape)."""
     with open(os.path.join(folder, "config.json"), "w") as f:
-        json.dump({"architecture": "Revitar", "vocab": REVITAR_VOCAB, "width": W,
-                   "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "residual_mult": 0.7,
-                   "layers": [one] * L}, f)
-    shapes = {"embed": (REVITAR_VOCAB, W), "head": (REVITAR_VOCAB, W), "final.norm": (W,)}
-    for i in range(L):
-        q = f"l{i}."
-        shapes.update({q + "norm1": (W,), q + "norm2": (W,), q + "mix.q": (H * D, W),
-                       q + "mix.k": (G * D, W), q + "mix.v": (G * D, W), q + "mix.o": (W, H * D),
-                       q + "mix.q.norm": (H * D,), q + "mix.k.norm": (G * D,), q + "mix.r1": (H,),
-                       q + "mix.r2": (H,), q + "mix.pb": (H,), q + "mlp.router": (E, W)})
-        for e in range(E):
-            shapes.update({f"{q}mlp.e{e}.gate": (ff, W), f"{q}mlp.e{e}.up": (ff, W),
-                           f"{q}mlp.e{e}.down": (W, ff)})
+        json.dump(config, f)
     header, at = {}, 0
     for name, sh in shapes.items():
         n = 2 * int(np.prod(sh))
@@ -635,17 +616,147 @@ def _write_revitar(torch, folder, size, layers=None):
     with open(os.path.join(folder, "model.safetensors"), "wb") as f:
         f.write(len(text).to_bytes(8, "little") + text)
         for name, sh in shapes.items():
-            t = torch.randn(sh, device="cuda", generator=g)
-            if name.endswith("norm") or "norm" in name.split(".")[-1]:
-                t = 1 + 0.1 * t
-            elif name.endswith((".r1", ".r2")):
-                t = 0.2 + 0.1 * t.abs()
-            elif name.endswith(".pb"):
-                t = t - 4
-            elif name != "embed":
-                t = t * sh[-1] ** -0.5
+            t = value(name, torch.randn(sh, device="cuda", generator=g), sh)
             f.write(t.to(torch.bfloat16).view(torch.int16).cpu().numpy().tobytes())
+
+
+def _write_revitar(torch, folder, size, layers=None):
+    """A Revitar model folder of that size with random bfloat16 weights; its parameter counts
+    [attention, router, one expert] per layer."""
+    W, H, G, D, window, E, top, ff, L = REVITAR_SIZES[size]
+    L = layers or L
+    one = {"type": "attention",
+           "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5,
+                     "softcap": 30.0, "mask": {"size": window}},
+           "mlp": {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": E, "top": top}}}
+    config = {"architecture": "Revitar", "vocab": REVITAR_VOCAB, "width": W,
+              "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6}, "residual_mult": 0.7,
+              "layers": [one] * L}
+    shapes = {"embed": (REVITAR_VOCAB, W), "head": (REVITAR_VOCAB, W), "final.norm": (W,)}
+    for i in range(L):
+        q = f"l{i}."
+        shapes.update({q + "norm1": (W,), q + "norm2": (W,), q + "mix.q": (H * D, W),
+                       q + "mix.k": (G * D, W), q + "mix.v": (G * D, W), q + "mix.o": (W, H * D),
+                       q + "mix.q.norm": (H * D,), q + "mix.k.norm": (G * D,), q + "mix.r1": (H,),
+                       q + "mix.r2": (H,), q + "mix.pb": (H,), q + "mlp.router": (E, W)})
+        for e in range(E):
+            shapes.update({f"{q}mlp.e{e}.gate": (ff, W), f"{q}mlp.e{e}.up": (ff, W),
+                           f"{q}mlp.e{e}.down": (W, ff)})
+
+    def value(name, t, sh):
+        if "norm" in name.split(".")[-1]:
+            return 1 + 0.1 * t
+        if name.endswith((".r1", ".r2")):
+            return 0.2 + 0.1 * t.abs()
+        return t - 4 if name.endswith(".pb") else t if name == "embed" else t * sh[-1] ** -0.5
+    _write_model(torch, folder, config, shapes, value)
     return [W * (2 * H * D + 2 * G * D), E * W, 3 * W * ff], L
+
+
+def _formats_agree(torch, kb, ctx, write):
+    """The number formats' logits on a small model of the class (a prompt in one portion, then token
+    by token): the median of their relative difference. Nothing is timed when they disagree."""
+    import tempfile
+    V, logits = REVITAR_VOCAB, []
+    with tempfile.TemporaryDirectory() as folder:
+        write(folder)
+        for compute in (kb.COMPUTE_BF16, kb.COMPUTE_F32):
+            mm = kb.Model.from_dir(ctx, folder, compute)
+            e = kb.Engine(mm, 512, 1)
+            toks = [int(t) for t in np.random.Generator(np.random.PCG64(1)).integers(0, V, 300)]
+            a = e.step([(1, toks[:280], list(range(0, 280, 9)))], V)
+            b = [e.step([(1, [t], [0])], V) for t in toks[280:]]
+            logits.append(np.concatenate([np.frombuffer(x, np.float32).reshape(-1, V)
+                                          for x in [a] + b]))
+            e.destroy()
+            mm.destroy()
+    d = np.sqrt(np.mean((logits[0] - logits[1]) ** 2, axis=1)) / np.std(logits[1])
+    if not np.median(d) <= 2e-2:
+        raise SystemExit(f"bench: bfloat16 and f32 logits differ by {np.median(d):.2e}")
+    return float(np.median(d))
+
+
+def _class_legs(torch, kb, ctx, stream, m, rng, ctx_len, flops, bytes_of, batches, only):
+    """Prompt and decode throughput of an unquantised model: one portion of 2048 tokens on 2048 cached
+    ones (`flops` of it), and the decode step at each batch with ctx_len tokens of context (`bytes_of`
+    a batch). `only`: that part once and untimed."""
+    hbm, tf, _ = _peaks()
+    V, bs, T, res = REVITAR_VOCAB, 16, 2048, {}
+    u = lambda x: np.ascontiguousarray(x, np.uint32)
+    dev = lambda x: torch.from_numpy(np.ascontiguousarray(x).astype(np.int32)).cuda()
+    if only != "decode":
+        # one prompt of 2 * T tokens in two portions; the second is timed
+        nb = (2 * T + bs - 1) // bs
+        pool = m.create_pool(nb, 1)
+        table, toks = u(rng.permutation(nb)), u(rng.integers(0, V, 2 * T))
+        logits = np.empty((1, V), np.float32)
+
+        def portion(start):
+            m.forward_step(pool, u(toks[start:start + T]), u([T]), u([start + T]), table, nb,
+                           u([T - 1]), logits)
+        portion(0)
+        for _ in range(1 if only else 3):
+            portion(T)
+        if not only:
+            l0 = ctx.launches
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record(stream)
+            for _ in range(5):
+                portion(T)
+            e1.record(stream)
+            torch.cuda.synchronize()
+            us = e0.elapsed_time(e1) * 1e3 / 5
+            res["prefill_2048_at_2048"] = {
+                "us": us, "tok/s": T / us * 1e6, "TFLOP/s": flops / us / 1e6,
+                "frac_of_tensor": flops / us / 1e6 / tf, "launches": int(ctx.launches - l0) // 5}
+        pool.destroy()
+    for B in () if only == "prefill" else batches:
+        c = ctx_len
+        nb = (c + bs - 1) // bs
+        pool = m.create_pool(nb * B, B)
+        tab = rng.permutation(nb * B).reshape(B, nb)
+        args = [dev(rng.integers(0, V, B)), dev(np.full(B, c - 1)),
+                dev(tab[:, -1] * bs + (c - 1) % bs), dev(tab), dev(np.full(B, c))]
+        logits = torch.empty(B, V, device="cuda")
+
+        def step():
+            m.decode_step_device(pool, *args, B, nb, c, logits)
+        l0 = ctx.launches
+        step()
+        ctx.sync()
+        launches = ctx.launches - l0
+        if not only:
+            us = _graph_time_us(torch, stream, step, 1)
+            ctx.sync()
+            byts = bytes_of(B)
+            res[f"decode_B{B}"] = {"us_per_step": us, "tok/s": B / us * 1e6,
+                                   "launches_per_step": int(launches), "alg_bytes": byts,
+                                   "GB/s": byts / us / 1e3, "frac_of_hbm": byts / us / 1e3 / hbm}
+        pool.destroy()
+    return res
+
+
+def _revitar_at(torch, kb, ctx, stream, size, batches, only=None, ctx_len=None):
+    """The legs of a Revitar model at one of REVITAR_SIZES."""
+    import tempfile
+    W, H, G, D, window, E, top, ff, _ = REVITAR_SIZES[size]
+    V, T = REVITAR_VOCAB, 2048
+    rng = np.random.Generator(np.random.PCG64(SEED + 71))
+    with tempfile.TemporaryDirectory() as folder:
+        (p_attn, p_router, p_expert), L = _write_revitar(torch, folder, size)
+        m = kb.Model.from_dir(ctx, folder)
+    c = ctx_len or min(4096, 2 * window)
+    keys = float(sum(min(window, T + i + 1) for i in range(T)))
+    flops = L * (2.0 * T * (p_attn + p_router + top * p_expert) + 4.0 * keys * H * D) + 2.0 * V * W
+
+    def bytes_of(B):
+        used = E * (1 - (1 - top / E) ** B)  # distinct experts, rows choosing at random
+        return (L * (2.0 * p_attn + 4 * p_router + 2 * used * p_expert +
+                     4.0 * B * min(window, c) * G * D) + 2.0 * V * W + 4.0 * B * V)
+    res = {"layers": L, **_class_legs(torch, kb, ctx, stream, m, rng, c, flops, bytes_of, batches,
+                                      only)}
+    m.destroy()
+    return res
 
 
 def revitar_legs(torch, kb, ctx, stream, sizes, batches=(1, 8, 32, 64), only=None):
@@ -656,101 +767,128 @@ def revitar_legs(torch, kb, ctx, stream, sizes, batches=(1, 8, 32, 64), only=Non
     decoding (weights of the chosen experts once, keys and values, logits), the tensor rate for
     prompts. `only`: "prefill" or "decode" of this class, or "llama" (the decode step beside it), once
     and untimed, for profiler captures."""
+    hbm, tf, src = _peaks()
+    out = {"peaks": {"hbm_GB/s": hbm, "bf16_TFLOP/s_sustained": tf, "source": src}}
+    for size in sizes:
+        W, H, G, D, window, E, top, ff, L = REVITAR_SIZES[size]
+        res = {"width": W, "heads": H, "kv_heads": G, "head": D, "window": window, "experts": E,
+               "top": top, "ff": ff}
+        if only == "llama":
+            out[size] = _llama_at(torch, kb, ctx, stream, size, L, batches, hbm, tf, once=True)
+            continue
+        if size == "1k" and not only:
+            res["check_bf16_vs_f32_median_rel_err"] = _formats_agree(
+                torch, kb, ctx, lambda folder: _write_revitar(torch, folder, size, layers=2))
+        res.update(_revitar_at(torch, kb, ctx, stream, size, batches, only))
+        if not only:
+            res["closest_q8_0_llama"] = _llama_at(torch, kb, ctx, stream, size, L, batches, hbm, tf)
+        out[size] = res
+    return out
+
+
+# Beside REVITAR_SIZES (width, experts, chosen experts, expert width and layers are theirs): heads,
+# unrotated, rotated and value columns of the latent attention, its two ranks; heads, key and value
+# columns of the matrix memory. Layers take turns; the first one's feed-forward is dense.
+MIGURAX_SIZES = {"1k": (16, 64, 32, 64, 256, 384, 4, 128, 256),
+                 "2k": (16, 128, 64, 128, 512, 768, 4, 256, 512),
+                 "4k": (32, 128, 64, 128, 512, 1536, 8, 256, 512)}
+
+
+def _write_migurax(torch, folder, size, layers=None):
+    """A Migurax model folder of that size with random bfloat16 weights; parameter counts {latent,
+    expand (of keys and values), memory, dense, router, expert} and the number of layers."""
+    W, _, _, _, _, E, top, ff, L = REVITAR_SIZES[size]
+    H, D, RD, DV, R, Q, MH, MD, MV = MIGURAX_SIZES[size]
+    V, L = REVITAR_VOCAB, layers or L
+    mixers = [{"heads": H, "dim": D, "rot_dim": RD, "vdim": DV, "kv_rank": R, "q_rank": Q,
+               "scale": (D + RD) ** -0.5, "rot": {"base": 10000.0, "dims": RD}},
+              {"heads": MH, "dim": MD, "vdim": MV, "gate_cap": 15.0}]
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": E, "top": top}}
+    config = {"architecture": "Migurax", "vocab": V, "width": W, "norm": {"eps": 1e-6},
+              "postln_alpha": 1.5,
+              "layers": [{"type": ("latent_attention", "mlstm")[i % 2], "mixer": mixers[i % 2],
+                          "mlp": moe if i else {"kind": "dense", "ff": top * ff}}
+                         for i in range(L)]}
+    shapes = {"embed": (V, W), "head": (V, W), "final.norm": (W,)}
+    for i in range(L):
+        p, x, q = f"l{i}.", f"l{i}.mix.", f"l{i}.mlp."
+        shapes.update({p + "norm1": (W,), p + "norm2": (W,)})
+        if i % 2 == 0:
+            shapes.update({x + "dq": (Q, W), x + "dq.norm": (Q,), x + "uq": (H * (D + RD), Q),
+                           x + "dkv": (R + RD, W), x + "dkv.norm": (R,), x + "uk": (H * D, R),
+                           x + "uv": (H * DV, R), x + "sink": (H,), x + "o": (W, H * DV)})
+        else:
+            shapes.update({x + "q": (MH * MD, W), x + "k": (MH * MD, W), x + "v": (MH * MV, W),
+                           x + "g": (MH * MV, W), x + "i": (MH, W), x + "f": (MH, W),
+                           x + "i.b": (MH,), x + "f.b": (MH,), x + "norm": (MH * MV,),
+                           x + "o": (W, MH * MV)})
+        if i == 0:
+            shapes.update({q + "up": (top * ff, W), q + "up.b": (top * ff,),
+                           q + "down": (W, top * ff), q + "down.b": (W,)})
+            continue
+        shapes.update({q + "router": (E, W), q + "router.b": (E,)})
+        for e in range(E):
+            shapes.update({f"{q}e{e}.up": (ff, W), f"{q}e{e}.down": (W, ff)})
+
+    def value(name, t, sh):
+        if "norm" in name.split(".")[-1]:
+            return 1 + 0.1 * t
+        if name.endswith(".f.b"):
+            return t + 4
+        return t if name == "embed" or len(sh) == 1 else t * sh[-1] ** -0.5
+    _write_model(torch, folder, config, shapes, value)
+    return {"latent": W * (Q + R + RD) + Q * H * (D + RD) + W * H * DV, "expand": R * H * (D + DV),
+            "memory": W * (2 * MH * MD + 2 * MH * MV + 2 * MH) + W * MH * MV,
+            "dense": 2 * W * top * ff, "router": E * W, "expert": 2 * W * ff}, L
+
+
+def migurax_legs(torch, kb, ctx, stream, sizes, batches=(1, 8, 32, 64), only=None):
+    """Prefill and decode of the Migurax class at real layer sizes (random weights), beside the closest
+    model of the library, a Revitar model with the same width, experts, layers and visible keys.
+    Fractions as in revitar_legs. Algorithmic work: for a prompt the cached latents expanded once to
+    keys and values, attention on those, and the matrix memory's update and read-out; for decoding
+    the weights, the cached latents, and each state read and written. `only`: "prefill" or "decode",
+    once and untimed; "revitar" (its decode step) and "revitar-prefill" likewise."""
     import tempfile
     hbm, tf, src = _peaks()
     out = {"peaks": {"hbm_GB/s": hbm, "bf16_TFLOP/s_sustained": tf, "source": src}}
     for size in sizes:
-        W, H, G, D, window, E, top, ff, _ = REVITAR_SIZES[size]
-        V, bs, T = REVITAR_VOCAB, 16, 2048
-        res = {"width": W, "heads": H, "kv_heads": G, "head": D, "window": window, "experts": E,
-               "top": top, "ff": ff}
-        rng = np.random.Generator(np.random.PCG64(SEED + 71))
-        if only == "llama":
-            out[size] = _llama_at(torch, kb, ctx, stream, size, REVITAR_SIZES[size][8], batches, hbm,
-                                  tf, once=True)
+        W, _, _, _, window, E, top, ff, _ = REVITAR_SIZES[size]
+        H, D, RD, DV, R, Q, MH, MD, MV = MIGURAX_SIZES[size]
+        V, T = REVITAR_VOCAB, 2048
+        if only and only.startswith("revitar"):
+            _revitar_at(torch, kb, ctx, stream, size, batches,
+                        "prefill" if only.endswith("prefill") else "decode", ctx_len=window)
             continue
+        res = {"width": W, "heads": H, "columns": [D, RD, DV], "ranks": [R, Q],
+               "memory": [MH, MD, MV], "experts": E, "top": top, "ff": ff, "context": window}
+        if size == "1k" and not only:
+            res["check_bf16_vs_f32_median_rel_err"] = _formats_agree(
+                torch, kb, ctx, lambda folder: _write_migurax(torch, folder, size, layers=3))
         with tempfile.TemporaryDirectory() as folder:
-            (p_attn, p_router, p_expert), L = _write_revitar(torch, folder, size)
+            n, L = _write_migurax(torch, folder, size)
             m = kb.Model.from_dir(ctx, folder)
         res["layers"] = L
-        if size == "1k" and not only:  # the number formats agree before anything is timed
-            with tempfile.TemporaryDirectory() as folder:
-                _write_revitar(torch, folder, size, layers=2)
-                logits = []
-                for compute in (kb.COMPUTE_BF16, kb.COMPUTE_F32):
-                    mm = kb.Model.from_dir(ctx, folder, compute)
-                    e = kb.Engine(mm, 512, 1)
-                    toks = [int(t) for t in np.random.Generator(np.random.PCG64(1)).integers(0, V, 300)]
-                    a = e.step([(1, toks[:280], list(range(0, 280, 9)))], V)
-                    b = [e.step([(1, [t], [0])], V) for t in toks[280:]]
-                    logits.append(np.concatenate([np.frombuffer(x, np.float32).reshape(-1, V)
-                                                  for x in [a] + b]))
-                    e.destroy()
-                    mm.destroy()
-            d = np.sqrt(np.mean((logits[0] - logits[1]) ** 2, axis=1)) / np.std(logits[1])
-            if not np.median(d) <= 2e-2:
-                raise SystemExit(f"bench: bfloat16 and f32 logits differ by {np.median(d):.2e}")
-            res["check_bf16_vs_f32_median_rel_err"] = float(np.median(d))
-        u = lambda x: np.ascontiguousarray(x, np.uint32)
-        dev = lambda x: torch.from_numpy(np.ascontiguousarray(x).astype(np.int32)).cuda()
-        if only != "decode":
-            # one prompt of 2 * T tokens in two portions; the second is timed
-            nb = (2 * T + bs - 1) // bs
-            pool = m.create_pool(nb)
-            table, toks = u(rng.permutation(nb)), u(rng.integers(0, V, 2 * T))
-            logits = np.empty((1, V), np.float32)
+        la, me, routed = (L + 1) // 2, L // 2, L - 1
+        pairs = float(sum(T + i + 1 for i in range(T)))
+        flops = (la * (2.0 * T * n["latent"] + 2.0 * 2 * T * n["expand"] +
+                       2.0 * pairs * H * (D + RD + DV)) +
+                 me * T * (2.0 * n["memory"] + 4.0 * MH * MD * MV) +
+                 2.0 * T * (n["dense"] + routed * (n["router"] + top * n["expert"])) + 2.0 * V * W)
+        state = 4.0 * MH * MV * MD
 
-            def portion(start):
-                m.forward_step(pool, u(toks[start:start + T]), u([T]), u([start + T]), table, nb,
-                               u([T - 1]), logits)
-            portion(0)
-            for _ in range(1 if only else 3):
-                portion(T)
-            if not only:
-                l0 = ctx.launches
-                e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-                e0.record(stream)
-                for _ in range(5):
-                    portion(T)
-                e1.record(stream)
-                torch.cuda.synchronize()
-                us = e0.elapsed_time(e1) * 1e3 / 5
-                keys = float(sum(min(window, T + i + 1) for i in range(T)))
-                flops = L * (2.0 * T * (p_attn + p_router + top * p_expert) + 4.0 * keys * H * D)
-                flops += 2.0 * V * W
-                res["prefill_2048_at_2048"] = {
-                    "us": us, "tok/s": T / us * 1e6, "TFLOP/s": flops / us / 1e6,
-                    "frac_of_tensor": flops / us / 1e6 / tf,
-                    "launches": int(ctx.launches - l0) // 5}
-            pool.destroy()
-        for B in () if only == "prefill" else batches:
-            c = min(4096, 2 * window)
-            nb = (c + bs - 1) // bs
-            pool = m.create_pool(nb * B)
-            tab = rng.permutation(nb * B).reshape(B, nb)
-            args = [dev(rng.integers(0, V, B)), dev(np.full(B, c - 1)),
-                    dev(tab[:, -1] * bs + (c - 1) % bs), dev(tab), dev(np.full(B, c))]
-            logits = torch.empty(B, V, device="cuda")
-
-            def step():
-                m.decode_step_device(pool, *args, B, nb, c, logits)
-            l0 = ctx.launches
-            step()
-            ctx.sync()
-            launches = ctx.launches - l0
-            if not only:
-                us = _graph_time_us(torch, stream, step, 1)
-                ctx.sync()
-                used = E * (1 - (1 - top / E) ** B)  # distinct experts, rows choosing at random
-                byts = (L * (2.0 * p_attn + 4 * p_router + 2 * used * p_expert +
-                             4.0 * B * min(window, c) * G * D) + 2.0 * V * W + 4.0 * B * V)
-                res[f"decode_B{B}"] = {"us_per_step": us, "tok/s": B / us * 1e6,
-                                       "launches_per_step": int(launches), "alg_bytes": byts,
-                                       "GB/s": byts / us / 1e3, "frac_of_hbm": byts / us / 1e3 / hbm}
-            pool.destroy()
+        def bytes_of(B):
+            used = E * (1 - (1 - top / E) ** B)  # distinct experts, rows choosing at random
+            return (la * (2.0 * (n["latent"] + n["expand"]) + 2.0 * B * window * (R + RD)) +
+                    me * (2.0 * n["memory"] + 2 * B * state) + 2.0 * n["dense"] +
+                    routed * (4 * n["router"] + 2 * used * n["expert"]) + 2.0 * V * W + 4.0 * B * V)
+        rng = np.random.Generator(np.random.PCG64(SEED + 73))
+        res.update(_class_legs(torch, kb, ctx, stream, m, rng, window, flops, bytes_of, batches,
+                               only))
         m.destroy()
         if not only:
-            res["closest_q8_0_llama"] = _llama_at(torch, kb, ctx, stream, size, L, batches, hbm, tf)
+            res["closest_revitar"] = _revitar_at(torch, kb, ctx, stream, size, batches,
+                                                 ctx_len=window)
         out[size] = res
     return out
 
@@ -1316,8 +1454,14 @@ def main():
                          f"({', '.join(REVITAR_SIZES)}) beside the Q8_0 llama step and print them")
     ap.add_argument("--revitar-only", default=None, metavar="prefill|decode[,B]|llama[,B]",
                     help="with --revitar: run that part once, untimed; for profiler captures")
+    ap.add_argument("--migurax", default=None, metavar="SIZE[,SIZE...]",
+                    help="time prefill and decode of the Migurax class at these sizes "
+                         f"({', '.join(MIGURAX_SIZES)}) beside the Revitar class and print them")
+    ap.add_argument("--migurax-only", default=None,
+                    metavar="prefill|decode[,B]|revitar[,B]|revitar-prefill",
+                    help="with --migurax: run that part once, untimed; for profiler captures")
     args = ap.parse_args()
-    if args.revitar:
+    if args.revitar or args.migurax:
         import torch
         kb = importlib.import_module("kanso-infer_b200").backend
         torch.cuda.set_device(0)
@@ -1325,9 +1469,11 @@ def main():
         torch.cuda.set_stream(stream)
         ctx = kb.Context(0, stream)
         ctx.set_option(kb.OPT_OVERLAP_WEIGHT_PREFETCH, 1)
-        only, _, b = (args.revitar_only or "").partition(",")
-        print(json.dumps(revitar_legs(torch, kb, ctx, stream, args.revitar.split(","),
-                                      (int(b),) if b else (1, 8, 32, 64), only or None)))
+        legs, sizes, what = (revitar_legs, args.revitar, args.revitar_only) if args.revitar else \
+            (migurax_legs, args.migurax, args.migurax_only)
+        only, _, b = (what or "").partition(",")
+        print(json.dumps(legs(torch, kb, ctx, stream, sizes.split(","),
+                              (int(b),) if b else (1, 8, 32, 64), only or None)))
         return
     if args.gemm_only:
         import torch

@@ -53,8 +53,9 @@ MODELS = {"attention": ATTENTION, "memory": MEMORY, "mixed": MIXED, "one": ONE, 
 
 def weights(cfg, seed):
     """Random tensors (float32, bfloat16 values). Queries are large, so that scores spread over
-    several units and single keys matter; the forget gates' biases spread from fading within a
-    few tokens to keeping hundreds."""
+    several units and single keys matter. In the matrix memory a token's query leans towards its own
+    key: a read-out next to zero is all rounding once its head's norm has made it one. The forget
+    gates' biases spread from fading within a few tokens to keeping hundreds."""
     rng = np.random.Generator(np.random.PCG64(seed))
     W, V = cfg["width"], cfg["vocab"]
     n = lambda *s, std=1.0: to_bf16(rng.standard_normal(s) * std)
@@ -67,7 +68,8 @@ def weights(cfg, seed):
         w[p + "norm1"] = near1(W)
         w[x + "o"] = lin(W, H * DV)
         if l["type"] == "mlstm":
-            w[x + "q"], w[x + "k"] = lin(H * D, W, 1.5), lin(H * D, W, 1.5)
+            w[x + "k"] = lin(H * D, W, 1.5)
+            w[x + "q"] = to_bf16(0.6 * w[x + "k"] + lin(H * D, W, 1.2))
             w[x + "v"], w[x + "g"] = lin(H * DV, W), lin(H * DV, W, 2.0)
             w[x + "i"], w[x + "f"] = lin(H, W, 1.5), lin(H, W, 1.0)
             w[x + "i.b"] = to_bf16(rng.uniform(-2, 2, H))
