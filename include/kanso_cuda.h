@@ -621,7 +621,8 @@ int32_t kanso_cuda_latent_store(kanso_cuda_ctx* ctx, kanso_cuda_kv* kv, uint32_t
 /* out f32[T][num_heads][rank] = sum_j softmax_j(scale * (q_lat . c_j + q_rot . k_rot_j)) c_j over the
  * keys at the row's position and before it. q_lat f32[T][num_heads][rank]; q f32[T][num_heads][dim +
  * rot], of which the last rot columns are rotated and used. path: 0 = the library's choice, 1 =
- * plain, 2 = mma.sync tiles (bfloat16; KANSO_ERR_UNSUPPORTED when a size is outside its range). */
+ * plain, 2 = mma.sync tiles (bfloat16, pages of 8, 16 or multiples of 32 tokens; KANSO_ERR_UNSUPPORTED
+ * when a size is outside its range). */
 int32_t kanso_cuda_latent_attention(kanso_cuda_ctx* ctx, const kanso_cuda_kv* kv, uint32_t layer,
                                     const float* q_lat, const float* q, const uint32_t* positions,
                                     const uint32_t* row_seq, const uint32_t* block_tables,

@@ -147,8 +147,9 @@ struct RowMap {
 enum class Residual : int { kAdd, kAddNorm };
 struct GemvSource {
   const float* x = nullptr;
-  int64_t x_ld = 0;     // row stride of x where there is no y (0: the columns)
-  int64_t x_group = 0;  // from one weight group's input to the next's
+  // Rows of x that lie further apart than the columns (not 0; without y), and from one weight
+  // group's input to the next's.
+  int64_t x_ld = 0, x_group = 0;
   float* x_out = nullptr;
   const float* y = nullptr;
   int parts = 1;
@@ -469,12 +470,12 @@ struct MlstmArgs {
 };
 // n portions, token by token from the state that earlier steps left. max_rows bounds their length.
 int32_t launch_mlstm_rows(kanso_cuda_ctx* ctx, const MlstmArgs& a, uint32_t n, uint32_t max_rows);
-// n portions in chunks of 64 tokens on the tensor cores; q, k, v are the bfloat16 operands. mem:
-// mlstm_chunk_bytes(a, T) of workspace.
+// n portions of at most max_rows tokens in chunks of 64 on the tensor cores; q, k, v are the bfloat16
+// operands. mem: mlstm_chunk_bytes of workspace for T, the rows of the step.
 bool mlstm_chunk_fits(const MlstmArgs& a);
 size_t mlstm_chunk_bytes(uint32_t heads, uint32_t dim, uint32_t vdim, int64_t T);
-int32_t launch_mlstm_chunks(kanso_cuda_ctx* ctx, const MlstmArgs& a, uint32_t n, void* mem,
-                            int64_t T);
+int32_t launch_mlstm_chunks(kanso_cuda_ctx* ctx, const MlstmArgs& a, uint32_t n, uint32_t max_rows,
+                            void* mem, int64_t T);
 // out[t] = each head of o over its own root mean square, times w, times sigmoid(gate), in the
 // products' element type; the gate lies in the projections' rows.
 int32_t launch_head_norm_gate(kanso_cuda_ctx* ctx, int32_t compute, const MlstmArgs& a,

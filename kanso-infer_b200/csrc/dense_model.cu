@@ -273,6 +273,7 @@ int32_t DenseModel::forward(kanso_cuda_kv* kv, const StepBatch& b, float* logits
     } else {
       const uint32_t base = (uint32_t)s.long_keys;
       longs.push_back({row, n, p0, i});
+      s.max_long_rows = std::max(s.max_long_rows, n);
       runs.push_back({base, c, i, 0});
       for (uint32_t k = 0; k < n; k += 128)
         long_tiles.push_back({row + k, std::min(128u, n - k), p0 + k, base});

@@ -34,7 +34,7 @@ struct DenseStep {
   // The sequences' portions, those shorter than PROMPT_MIN_ROWS first. nullptr: row t is all of
   // sequence t.
   const AttnTile* portions = nullptr;
-  uint32_t n_short = 0, n_long = 0, max_short_rows = 1;
+  uint32_t n_short = 0, n_long = 0, max_short_rows = 1, max_long_rows = 0;
   const uint32_t* short_rows = nullptr;  // the rows of short portions (nullptr: every row)
   int64_t n_short_rows = 0;
   // Long portions in tiles of 128 rows whose last word is where the sequence's keys begin when

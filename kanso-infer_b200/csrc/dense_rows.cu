@@ -472,30 +472,52 @@ __global__ void __launch_bounds__(DR_THREADS)
 }
 
 // ---- matrix memory: the heads' outputs on the way to the o-projection ----
+// One CTA per head and row.
+constexpr int HN_THREADS = 128;
 template <typename E>
-__global__ void __launch_bounds__(DR_THREADS)
+__global__ void __launch_bounds__(HN_THREADS)
     head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ gate,
                           int64_t gate_ld, int parts, int64_t part_stride, int heads, int hd,
                           const float* __restrict__ w, float eps, E* __restrict__ out,
                           int64_t out_ld) {
+  __shared__ float red[32];
   pdl_launch_dependents();
   pdl_wait();
-  const int64_t t = blockIdx.x;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = heads * hd;
-  const float *x = o + t * n, *g = gate + t * gate_ld;
-  for (int h = warp; h < heads; h += DR_THREADS / 32) {
-    float ss = 0.f;
-    for (int i = lane; i < hd; i += 32) ss += x[h * hd + i] * x[h * hd + i];
-#pragma unroll
-    for (int s = 16; s; s >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, s);
+  const int h = blockIdx.x, n = heads * hd;
+  const int64_t t = blockIdx.y;
+  const float *x = o + t * n + h * hd, *g = gate + t * gate_ld + h * hd;
+  E* dst = out + t * out_ld + h * hd;
+  w += h * hd;
+  float ss = 0.f;
+  if (hd % 4 == 0 && gate_ld % 4 == 0 && part_stride % 4 == 0 &&
+      ((reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & 15u) == 0 &&
+      out_ld % 4 == 0) {
+    for (int i = threadIdx.x * 4; i < hd; i += HN_THREADS * 4)
+      ss += sum_sq4(*reinterpret_cast<const float4*>(x + i));
+    ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)hd + eps);
-    for (int i = h * hd + lane; i < (h + 1) * hd; i += 32) {
+    for (int i = threadIdx.x * 4; i < hd; i += HN_THREADS * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(x + i);
+      const float4 k = *reinterpret_cast<const float4*>(w + i);
+      float4 z = *reinterpret_cast<const float4*>(g + i);
+#pragma unroll 3
+      for (int p = 1; p < parts; ++p)
+        add4(z, *reinterpret_cast<const float4*>(g + p * part_stride + i));
+      store4(dst + i, v.x * inv * k.x / (1.0f + expf(-z.x)), v.y * inv * k.y / (1.0f + expf(-z.y)),
+             v.z * inv * k.z / (1.0f + expf(-z.z)), v.w * inv * k.w / (1.0f + expf(-z.w)));
+    }
+  } else {
+    for (int i = threadIdx.x; i < hd; i += HN_THREADS) ss += x[i] * x[i];
+    ss = block_sum(ss, red);
+    const float inv = 1.0f / sqrtf(ss / (float)hd + eps);
+    for (int i = threadIdx.x; i < hd; i += HN_THREADS) {
       float z = g[i];
       for (int p = 1; p < parts; ++p) z += g[p * part_stride + i];
-      out[t * out_ld + i] = to_elem<E>(x[i] * inv * w[i] / (1.0f + expf(-z)));
+      dst[i] = to_elem<E>(x[i] * inv * w[i] / (1.0f + expf(-z)));
     }
   }
-  for (int i = n + threadIdx.x; i < out_ld; i += DR_THREADS) out[t * out_ld + i] = to_elem<E>(0.f);
+  if (h == heads - 1)
+    for (int i = n + threadIdx.x; i < out_ld; i += HN_THREADS) out[t * out_ld + i] = to_elem<E>(0.f);
 }
 
 #define DR_LAUNCH(kern, grid, threads, smem, what, ...)                                          \
@@ -649,11 +671,17 @@ int32_t launch_head_norm_gate(kanso_cuda_ctx* ctx, int32_t compute, const MlstmA
                               const float* w, float eps, void* out, int64_t out_ld, int64_t T) {
   const int H = a.heads, V = a.vdim;
   const float* gate = a.y + (int64_t)H * (2 * a.dim + V);
-  if (compute == KANSO_COMPUTE_BF16)
-    DR_LAUNCH(head_norm_gate_kernel<bf16>, T, DR_THREADS, 0, "head_norm_gate", a.out, gate,
-              a.width(), a.parts, a.part_stride, H, V, w, eps, (bf16*)out, out_ld);
-  DR_LAUNCH(head_norm_gate_kernel<float>, T, DR_THREADS, 0, "head_norm_gate", a.out, gate,
-            a.width(), a.parts, a.part_stride, H, V, w, eps, (float*)out, out_ld);
+  const dim3 grid((unsigned)H, (unsigned)T);
+  const cudaError_t e =
+      compute == KANSO_COMPUTE_BF16
+          ? launch_dependent(ctx, head_norm_gate_kernel<bf16>, grid, dim3(HN_THREADS), 0, a.out,
+                             gate, a.width(), a.parts, a.part_stride, H, V, w, eps, (bf16*)out,
+                             out_ld)
+          : launch_dependent(ctx, head_norm_gate_kernel<float>, grid, dim3(HN_THREADS), 0, a.out,
+                             gate, a.width(), a.parts, a.part_stride, H, V, w, eps, (float*)out,
+                             out_ld);
+  if (e != cudaSuccess) return cuda_fail(ctx, e, "head_norm_gate");
+  return after_launch(ctx, "head_norm_gate");
 }
 
 }  // namespace kanso

@@ -40,15 +40,24 @@ struct GemmDenseArgs {
   const uint32_t* row_list;
   int relu2, elem, n_end;  // n_end: columns that are written
 
-  __device__ __forceinline__ float finish(float v, int n) const {
-    if (bias && n < rows && blockIdx.z == 0) v += bias[n];
-    return relu2 ? relu_squared(v) : v;
+  // The bias of column n, added once where the columns' sum is split.
+  __device__ __forceinline__ float bias_of(int n) const {
+    return bias && n < rows && blockIdx.z == 0 ? bias[n] : 0.f;
   }
-  // Element offset of a result row.
-  __device__ __forceinline__ int64_t row_at(int64_t row, int group) const {
-    if (!group_step) return row * out_ld;
-    const int64_t r = row - group * (T / groups);
-    return (row_list ? row_list[r] : r) * out_ld + group * group_step;
+};
+// Where the rows of a tile's group go: row r at r * out_ld + shift, by the list if there is one.
+struct RowPlace {
+  int64_t shift = 0, first = 0;
+  const uint32_t* list = nullptr;
+  __device__ __forceinline__ RowPlace(const GemmDenseArgs& a, int group) {
+    if (!a.group_step) return;
+    const int64_t per = (uint32_t)a.T / (uint32_t)a.groups;
+    shift = group * (a.row_list ? a.group_step : a.group_step - per * a.out_ld);
+    first = group * per;
+    list = a.row_list;
+  }
+  __device__ __forceinline__ int64_t at(int64_t row, int64_t out_ld) const {
+    return (list ? (int64_t)list[row - first] : row) * out_ld + shift;
   }
 };
 
@@ -57,11 +66,18 @@ __device__ __forceinline__ bool find_tile(const uint32_t* offsets, int groups, i
                                           int tile, int lane, int* group, int64_t* first,
                                           int64_t* end) {
   if (!offsets) {
-    const int64_t per = T / groups, tiles = (per + nt - 1) / nt;
-    *group = (int)(tile / tiles);
-    *first = *group * per + tile % tiles * nt;
-    *end = (*group + 1) * per;
-    return *group < groups;
+    if (groups == 1) {
+      *group = 0;
+      *first = (int64_t)tile * nt;
+      *end = T;
+      return *first < T;
+    }
+    const uint32_t per = (uint32_t)T / (uint32_t)groups, tiles = (per + nt - 1) / (uint32_t)nt;
+    const uint32_t g = (uint32_t)tile / tiles;
+    *group = (int)g;
+    *first = (int64_t)g * per + (int64_t)((uint32_t)tile - g * tiles) * nt;
+    *end = (int64_t)(g + 1) * per;
+    return g < (uint32_t)groups;
   }
   int before = 0;
   for (int g0 = 0; g0 < groups; g0 += 32) {
@@ -209,34 +225,44 @@ __global__ void __launch_bounds__(GD_THREADS)
     const int n = n0 + warp * 32 + lane;  // a warp reaches its own quarter of the TMEM lanes
     const uint32_t lane_base = tmem + ((uint32_t)(warp * 32) << 16);
     const int valid = (int)min((int64_t)NT, tile_end - tile_first);
+    const RowPlace place(a, tile_group);
+    const float b0 = a.bias_of(n), b1 = DUAL ? a.bias_of(n + 128) : 0.f;
+    const bool in0 = n < a.n_end, in1 = n + 128 < a.n_end;
     for (int c = 0; c < NT / 16; ++c) {
       if (c * 16 >= valid) break;
       uint32_t r0[16], r1[16];
       tmem_ld16(lane_base + c * 16, r0);
       if (DUAL) tmem_ld16(lane_base + NT + c * 16, r1);
+      if (ACT) {
 #pragma unroll
-      for (int j = 0; j < 16; ++j) {
-        const int m = c * 16 + j;
-        if (m >= valid) continue;
-        const int64_t row = tile_first + m;
-        if (ACT) {
+        for (int j = 0; j < 16; ++j) {
+          if (c * 16 + j >= valid) continue;
           // the pad columns multiply weight rows that were zero-filled: they come out as zero
           const float g = __uint_as_float(r0[j]), u = __uint_as_float(r1[j]);
           if (n < a.out_ld)
-            static_cast<bf16*>(a.out)[row * a.out_ld + n] = to_elem<bf16>(silu(g) * u);
-        } else {
-          const int64_t at = (int64_t)blockIdx.z * a.part_stride + a.row_at(row, tile_group);
-          const float v0 = a.finish(__uint_as_float(r0[j]), n);
-          const float v1 = DUAL ? a.finish(__uint_as_float(r1[j]), n + 128) : 0.f;
-          if (a.elem) {
-            bf16* o = static_cast<bf16*>(a.out) + at;
-            if (n < a.n_end) o[n] = to_elem<bf16>(v0);
-            if (DUAL && n + 128 < a.n_end) o[n + 128] = to_elem<bf16>(v1);
-          } else {
-            float* o = static_cast<float*>(a.out) + at;
-            if (n < a.n_end) o[n] = v0;
-            if (DUAL && n + 128 < a.n_end) o[n + 128] = v1;
-          }
+            static_cast<bf16*>(a.out)[(tile_first + c * 16 + j) * a.out_ld + n] =
+                to_elem<bf16>(silu(g) * u);
+        }
+      } else if (a.elem) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+          if (c * 16 + j >= valid) continue;
+          float v0 = __uint_as_float(r0[j]) + b0, v1 = DUAL ? __uint_as_float(r1[j]) + b1 : 0.f;
+          if (a.relu2) v0 = relu_squared(v0), v1 = relu_squared(v1);
+          bf16* o = static_cast<bf16*>(a.out) + place.at(tile_first + c * 16 + j, a.out_ld) + n;
+          if (in0) o[0] = to_elem<bf16>(v0);
+          if (DUAL && in1) o[128] = to_elem<bf16>(v1);
+        }
+      } else {
+        float* part = static_cast<float*>(a.out) + (int64_t)blockIdx.z * a.part_stride + n;
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+          if (c * 16 + j >= valid) continue;
+          float v0 = __uint_as_float(r0[j]) + b0, v1 = DUAL ? __uint_as_float(r1[j]) + b1 : 0.f;
+          if (a.relu2) v0 = relu_squared(v0), v1 = relu_squared(v1);
+          float* o = part + place.at(tile_first + c * 16 + j, a.out_ld);
+          if (in0) o[0] = v0;
+          if (DUAL && in1) o[128] = v1;
         }
       }
     }
@@ -312,6 +338,7 @@ __global__ void __launch_bounds__(256)
         }
     }
   }
+  const RowPlace place(a, tile_group);
 #pragma unroll
   for (int m = 0; m < 4; ++m) {
     const int64_t row = tile_first + ty + 16 * m;
@@ -319,9 +346,13 @@ __global__ void __launch_bounds__(256)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int n = n0 + tx + 16 * i;
-      if (n < (ACT ? a.out_ld : a.n_end))
-        static_cast<float*>(a.out)[a.row_at(row, tile_group) + n] =
-            ACT ? silu(acc[m][i]) * acu[m][i] : a.finish(acc[m][i], n);
+      if (ACT) {
+        if (n < a.out_ld)
+          static_cast<float*>(a.out)[row * a.out_ld + n] = silu(acc[m][i]) * acu[m][i];
+      } else if (n < a.n_end) {
+        const float v = acc[m][i] + a.bias_of(n);
+        static_cast<float*>(a.out)[place.at(row, a.out_ld) + n] = a.relu2 ? relu_squared(v) : v;
+      }
     }
   }
 }

@@ -115,6 +115,10 @@ __device__ __forceinline__ void finish_rows(float (&acc)[V], int ks, float* red,
   __syncthreads();
 }
 
+// What a launch of the plain product's kernel is made for: rows with the residual step, inputs that
+// lie in groups (and the store beside them), or gated heads.
+enum GemvKind { GV_ROWS_IN, GV_GROUPS_IN, GV_GATED_IN };
+
 struct GemvArgs {
   const void* w;
   int rows, cols, ld, ks, T;
@@ -147,51 +151,51 @@ __device__ __forceinline__ void gate_source(const GemvSource& s, const float* x,
   }
 }
 
-// The residual step for the rows of this CTA, into shared memory (and to x_out by one CTA).
-template <int TT>
+// The input rows of this CTA, into shared memory (and the residual step's to x_out by one CTA).
+template <int TT, int KIND>
 __device__ __forceinline__ void norm_source(const GemvSource& s, int cols, int ld, int t0, int nt,
                                             bool writer, float* xs, float* red) {
   for (int t = 0; t < nt; ++t) {
     const int64_t r = s.row_index ? s.row_index[t0 + t] : t0 + t;
-    const float* y = s.y + r * cols;
-    const float* x = s.x + r * (s.x_ld ? s.x_ld : cols) + blockIdx.z * s.x_group;
+    const float* x = s.x + r * cols;
     float* xt = xs + t * ld;
-    const bool after = s.form == Residual::kAddNorm;
-    if (s.gate) {
+    if (KIND == GV_GATED_IN) {
       gate_source(s, x, s.gate + r * s.gate_ld, cols, ld, xt);
-      for (int i = cols + threadIdx.x; i < ld; i += GV_THREADS) xt[xs_index(i, ld)] = 0.f;
-      continue;
-    }
-    float ss = 0.f;
-    if (s.y) {
+    } else {
+      if (KIND == GV_GROUPS_IN) x = s.x + r * s.x_ld + blockIdx.z * s.x_group;
+      const bool step = KIND == GV_ROWS_IN && s.y;
+      const bool after = step && s.form == Residual::kAddNorm;
+      float inv = 0.f;
+      if (step) {
+        const float* y = s.y + r * cols;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < cols; i += GV_THREADS) {
+          float v = y[i];
+          for (int p = 1; p < s.parts; ++p) v += y[p * s.part_stride + i];
+          if (after) v = fmaf(s.mult, x[i], v);
+          xt[xs_index(i, ld)] = v;
+          ss += v * v;
+        }
+        ss = block_sum(ss, red);
+        inv = 1.0f / sqrtf(ss / (float)cols + s.eps);
+      }
+      float s2 = 0.f;
       for (int i = threadIdx.x; i < cols; i += GV_THREADS) {
-        float v = y[i];
-        for (int p = 1; p < s.parts; ++p) v += y[p * s.part_stride + i];
-        if (after) v = fmaf(s.mult, x[i], v);
+        float v = after ? 0.f : x[i];
+        if (step) {
+          const float n = xt[xs_index(i, ld)] * inv * s.norm_w[i];
+          v = after ? n : v + s.mult * n;
+        }
         xt[xs_index(i, ld)] = v;
-        ss += v * v;
+        if (writer && s.x_out) s.x_out[r * cols + i] = v;
+        s2 += v * v;
       }
-      ss = block_sum(ss, red);
-    }
-    const float inv = s.y ? 1.0f / sqrtf(ss / (float)cols + s.eps) : 0.f;
-    float s2 = 0.f;
-    for (int i = threadIdx.x; i < cols; i += GV_THREADS) {
-      float v;
-      if (s.y && after) {
-        v = xt[xs_index(i, ld)] * inv * s.norm_w[i];
-      } else {
-        v = x[i];
-        if (s.y) v += s.mult * (xt[xs_index(i, ld)] * inv * s.norm_w[i]);
+      if (s.final_w) {
+        s2 = block_sum(s2, red);
+        const float inv2 = 1.0f / sqrtf(s2 / (float)cols + s.eps);
+        for (int i = threadIdx.x; i < cols; i += GV_THREADS)
+          xt[xs_index(i, ld)] = xt[xs_index(i, ld)] * inv2 * s.final_w[i];
       }
-      xt[xs_index(i, ld)] = v;
-      if (writer && s.x_out) s.x_out[r * cols + i] = v;
-      s2 += v * v;
-    }
-    if (s.final_w) {
-      s2 = block_sum(s2, red);
-      const float inv2 = 1.0f / sqrtf(s2 / (float)cols + s.eps);
-      for (int i = threadIdx.x; i < cols; i += GV_THREADS)
-        xt[xs_index(i, ld)] = xt[xs_index(i, ld)] * inv2 * s.final_w[i];
     }
     for (int i = cols + threadIdx.x; i < ld; i += GV_THREADS) xt[xs_index(i, ld)] = 0.f;
   }
@@ -199,23 +203,30 @@ __device__ __forceinline__ void norm_source(const GemvSource& s, int cols, int l
     for (int i = threadIdx.x; i < ld; i += GV_THREADS) xs[t * ld + i] = 0.f;
 }
 
-template <typename E, int TT>
-__global__ void __launch_bounds__(GV_THREADS) gemv_dense_kernel(const GemvArgs a) {
+template <typename E, int TT, int KIND>
+__global__ void __launch_bounds__(GV_THREADS, sizeof(E) == 2 ? (TT == 1 ? 4 : 3) : 2)
+    gemv_dense_kernel(const GemvArgs a) {
   extern __shared__ __align__(16) float xs[];
   __shared__ float red[GV_WARPS * GV_ROWS * TT > 32 ? GV_WARPS * GV_ROWS * TT : 32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int gpc = GV_WARPS / a.ks, sub = warp % a.ks, chunks = a.ld / 8;
   const int t0 = blockIdx.y * TT, nt = min(TT, a.T - t0);
   const int groups = (a.rows + GV_ROWS - 1) / GV_ROWS;
-  if ((int)blockIdx.x < a.store_ctas) {
-    pdl_launch_dependents();
-    pdl_wait();
-    if (blockIdx.y == 0 && blockIdx.z == 0) latent_store_row<E>(a.store, blockIdx.x, red);
-    return;
+  const E* w = static_cast<const E*>(a.w);
+  float* out = a.out;
+  int cta = blockIdx.x, ctas = gridDim.x;
+  if (KIND == GV_GROUPS_IN) {
+    if (cta < a.store_ctas) {
+      pdl_launch_dependents();
+      pdl_wait();
+      if (blockIdx.y == 0 && blockIdx.z == 0) latent_store_row<E>(a.store, cta, red);
+      return;
+    }
+    cta -= a.store_ctas;
+    ctas -= a.store_ctas;
+    w += (int64_t)blockIdx.z * a.rows * a.ld;
+    out += blockIdx.z * a.o.group_step;
   }
-  const int cta = blockIdx.x - a.store_ctas, ctas = gridDim.x - a.store_ctas;
-  const E* w = static_cast<const E*>(a.w) + (int64_t)blockIdx.z * a.rows * a.ld;
-  float* out = a.out + blockIdx.z * a.o.group_step;
   const int c0 = sub * 32 + lane, step = a.ks * 32;
   const E* row[GV_ROWS];
   RawOf<E> cur[GV_ROWS];
@@ -230,7 +241,7 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_dense_kernel(const GemvArgs a
   open_group(base + warp / a.ks);  // weights depend on nothing that runs before this kernel
   pdl_launch_dependents();
   pdl_wait();
-  norm_source<TT>(a.s, a.cols, a.ld, t0, nt, cta == 0 && blockIdx.z == 0, xs, red);
+  norm_source<TT, KIND>(a.s, a.cols, a.ld, t0, nt, cta == 0, xs, red);
   __syncthreads();
   while (true) {
     float acc[GV_ROWS * TT];
@@ -405,14 +416,20 @@ static unsigned gv_grid(const kanso_cuda_ctx* ctx, int64_t groups, int ks, int64
   return (unsigned)std::min(need, cap);
 }
 
-template <typename E, int TT>
+template <typename E, int TT, int KIND>
 static int32_t gemv_launch(kanso_cuda_ctx* ctx, const GemvArgs& a, dim3 grid, size_t smem) {
-  int32_t st = allow_max_smem(ctx, (const void*)gemv_dense_kernel<E, TT>);
+  int32_t st = allow_max_smem(ctx, (const void*)gemv_dense_kernel<E, TT, KIND>);
   if (st) return st;
   const cudaError_t e =
-      launch_dependent(ctx, gemv_dense_kernel<E, TT>, grid, dim3(GV_THREADS), smem, a);
+      launch_dependent(ctx, gemv_dense_kernel<E, TT, KIND>, grid, dim3(GV_THREADS), smem, a);
   if (e != cudaSuccess) return cuda_fail(ctx, e, "gemv_dense launch");
   return after_launch(ctx, "gemv_dense");
+}
+template <typename E, int TT>
+static int32_t gemv_launch(kanso_cuda_ctx* ctx, const GemvArgs& a, dim3 grid, size_t smem) {
+  if (a.s.gate) return gemv_launch<E, TT, GV_GATED_IN>(ctx, a, grid, smem);
+  if (a.s.x_ld) return gemv_launch<E, TT, GV_GROUPS_IN>(ctx, a, grid, smem);
+  return gemv_launch<E, TT, GV_ROWS_IN>(ctx, a, grid, smem);
 }
 
 int32_t launch_gemv(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat& w, const GemvSource& s,
@@ -424,7 +441,7 @@ int32_t launch_gemv(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat& w, con
     return fail(ctx, KANSO_ERR_UNSUPPORTED, "dense product: %lld columns", (long long)w.cols);
   const int64_t groups = (w.rows + GV_ROWS - 1) / GV_ROWS, copies = (T + tt - 1) / tt;
   const int64_t all = copies * w.groups;
-  if (w.groups > 65535)
+  if (w.groups > 65535 || ((w.groups > 1 || store) && (!s.x_ld || s.y)))
     return fail(ctx, KANSO_ERR_UNSUPPORTED, "dense product: %lld groups", (long long)w.groups);
   GemvArgs a = {w.w, (int)w.rows, (int)w.cols, (int)w.ld, pick_ks(ctx, groups, all, w.ld / 8),
                 T, s, out, out_ld, o, store ? T : 0, store ? *store : LatentStore()};

@@ -7,13 +7,15 @@
 //   out = sum_j exp(s_j) c_j / (sum_j exp(s_j) + exp(sink))
 //
 // latent_rows: four heads per CTA, any size, f32 and (sizes beyond the other) bfloat16.
-// latent_group: bfloat16, sixteen heads as the rows of an mma tile, 64 keys at a time; a staged row
-// serves as key and as value. A row's keys may be shared out over several CTAs: partial sums with
-// their maxima are merged in order by the CTA that arrives last.
+// latent_group: bfloat16, sixteen heads as the rows of an mma tile, 32 keys at a time; a staged row
+// serves as key and as value. A row's keys may be shared out over several CTAs, which leave partial
+// sums with their maxima; latent_merge adds them in order.
 #include <algorithm>
 #include <cmath>
 
 #include "dense.cuh"
+#include "tc05.cuh"
+#include "tensor_map.h"
 #include "warp_mma.cuh"
 
 namespace kanso {
@@ -22,9 +24,9 @@ struct LatentRowsArgs {
   LatentAttn a;
   KvDenseLayer kv;
   LatentRows r;
-  float* partial;   // [n][heads][parts][rank + 2]: sums, maximum, denominator
-  uint32_t* tickets;
-  uint32_t parts, tile;
+  float* partial;  // parts > 1: [n][heads][parts][rec]: sums, maximum, denominator
+  uint32_t parts, tile, rec;
+  int stages;
   int* status;
 };
 
@@ -53,36 +55,58 @@ __device__ __forceinline__ float latent_q_value(const LatentQuery& q, int64_t at
   for (int p = 1; p < q.parts; ++p) v += q.q[p * q.part_stride + at];
   return v;
 }
-// The shares of heads [h0, h0 + nh) of row i, and the store of the result. All threads.
 template <typename E>
-__device__ __forceinline__ void latent_merge(const LatentRowsArgs& p, int64_t i, int h0, int nh,
-                                             uint32_t n_parts, float* coef) {
-  const int R = p.a.rank;
-  const size_t rec = (size_t)R + 2;
-  const float* src = p.partial + ((size_t)i * p.a.heads + h0) * p.parts * rec;
-  for (int h = threadIdx.x; h < nh; h += blockDim.x) {
-    const float* m = src + (size_t)h * p.parts * rec + R;
-    const float sink = p.a.sink[h0 + h];
+__device__ __forceinline__ void latent_out(const LatentRowsArgs& p, int64_t i, int h, int c,
+                                           float v) {
+  const int64_t at = i * p.r.out_row + h * p.r.out_head + c;
+  if (p.r.out_f32)
+    static_cast<float*>(p.r.out)[at] = v;
+  else
+    static_cast<E*>(p.r.out)[at] = to_elem<E>(v);
+}
+
+// The shares of one head of one row (blockIdx.x, blockIdx.y), four columns per thread.
+constexpr int LM_THREADS = 128;
+template <typename E>
+__global__ void __launch_bounds__(LM_THREADS) latent_merge_kernel(const LatentRowsArgs p) {
+  extern __shared__ float weight[];  // [parts]
+  pdl_launch_dependents();
+  const int h = blockIdx.x, R = p.a.rank;
+  const int64_t i = blockIdx.y;
+  const uint32_t n = latent_span(p, i, 0).n_parts;
+  const float* src = p.partial + ((size_t)i * p.a.heads + h) * p.parts * p.rec;
+  pdl_wait();
+  if (threadIdx.x < 32) {
+    const float sink = p.a.sink[h];
     float top = sink, den = 0.f;
-    for (uint32_t k = 0; k < n_parts; ++k) top = fmaxf(top, __ldcg(m + k * rec));
-    for (uint32_t k = 0; k < n_parts; ++k)
-      den += __ldcg(m + k * rec + 1) * expf(__ldcg(m + k * rec) - top);
-    coef[2 * h] = top;
-    coef[2 * h + 1] = 1.0f / (den + expf(sink - top));
+    for (uint32_t k = threadIdx.x; k < n; k += 32)
+      top = fmaxf(top, src[(size_t)k * p.rec + p.rec - 4]);
+#pragma unroll
+    for (int o = 16; o; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xFFFFFFFFu, top, o));
+    for (uint32_t k = threadIdx.x; k < n; k += 32) {
+      const float w = expf(src[(size_t)k * p.rec + p.rec - 4] - top);
+      den += w * src[(size_t)k * p.rec + p.rec - 3];
+      weight[k] = w;
+    }
+#pragma unroll
+    for (int o = 16; o; o >>= 1) den += __shfl_xor_sync(0xFFFFFFFFu, den, o);
+    const float inv = 1.0f / (den + expf(sink - top));
+    for (uint32_t k = threadIdx.x; k < n; k += 32) weight[k] *= inv;
   }
   __syncthreads();
-  for (int k = threadIdx.x; k < nh * R; k += blockDim.x) {
-    const int h = k / R, c = k - h * R;
-    const float* o = src + (size_t)h * p.parts * rec;
-    float v = 0.f;
-    for (uint32_t s = 0; s < n_parts; ++s)
-      v += __ldcg(o + s * rec + c) * expf(__ldcg(o + s * rec + R) - coef[2 * h]);
-    v *= coef[2 * h + 1];
-    const int64_t at = i * p.r.out_row + (h0 + h) * p.r.out_head + c;
-    if (p.r.out_f32)
-      static_cast<float*>(p.r.out)[at] = v;
-    else
-      static_cast<E*>(p.r.out)[at] = to_elem<E>(v);
+  for (int c = threadIdx.x * 4; c < R; c += LM_THREADS * 4) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (uint32_t k = 0; k < n; ++k) {
+      const float4 o = *reinterpret_cast<const float4*>(src + (size_t)k * p.rec + c);
+      const float w = weight[k];
+      v.x = fmaf(w, o.x, v.x), v.y = fmaf(w, o.y, v.y);
+      v.z = fmaf(w, o.z, v.z), v.w = fmaf(w, o.w, v.w);
+    }
+    latent_out<E>(p, i, h, c, v.x);
+    if (c + 1 < R) latent_out<E>(p, i, h, c + 1, v.y);
+    if (c + 2 < R) latent_out<E>(p, i, h, c + 2, v.z);
+    if (c + 3 < R) latent_out<E>(p, i, h, c + 3, v.w);
   }
 }
 
@@ -92,9 +116,8 @@ constexpr int LR_THREADS = 128, LR_HEADS = 4, LR_TILE = 32;
 template <typename E>
 __global__ void __launch_bounds__(LR_THREADS) latent_rows_kernel(const LatentRowsArgs p) {
   extern __shared__ __align__(16) float sm[];
-  __shared__ float prob[LR_HEADS][LR_TILE], corr[LR_HEADS], coef[2 * LR_HEADS];
+  __shared__ float prob[LR_HEADS][LR_TILE], corr[LR_HEADS];
   __shared__ size_t key_at[LR_TILE];
-  __shared__ uint32_t ticket;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int part = blockIdx.x, h0 = blockIdx.y * LR_HEADS;
   const int64_t i = blockIdx.z;
@@ -184,7 +207,7 @@ __global__ void __launch_bounds__(LR_THREADS) latent_rows_kernel(const LatentRow
     }
   }
   __syncthreads();
-  if (s.n_parts == 1) {
+  if (p.parts == 1) {
     if (lane == 0 && warp < nh) {
       const float sink = p.a.sink[h0 + warp], top = fmaxf(m, sink), c = expf(m - top);
       corr[warp] = c / (l * c + expf(sink - top));
@@ -192,115 +215,150 @@ __global__ void __launch_bounds__(LR_THREADS) latent_rows_kernel(const LatentRow
     __syncthreads();
     for (int k = tid; k < nh * R; k += LR_THREADS) {
       const int h = k / R, c = k - h * R;
-      const float v = acc[h * KL + c] * corr[h];
-      const int64_t at = i * p.r.out_row + (h0 + h) * p.r.out_head + c;
-      if (p.r.out_f32)
-        static_cast<float*>(p.r.out)[at] = v;
-      else
-        static_cast<E*>(p.r.out)[at] = to_elem<E>(v);
+      latent_out<E>(p, i, h0 + h, c, acc[h * KL + c] * corr[h]);
     }
     return;
   }
-  const size_t rec = (size_t)R + 2;
-  float* mine = p.partial + ((size_t)i * H + h0) * p.parts * rec + part * rec;
+  float* mine = p.partial + (((size_t)i * H + h0) * p.parts + part) * p.rec;
+  const size_t head = (size_t)p.parts * p.rec;
   for (int k = tid; k < nh * R; k += LR_THREADS) {
     const int h = k / R, c = k - h * R;
-    mine[(size_t)h * p.parts * rec + c] = acc[h * KL + c];
+    mine[h * head + c] = acc[h * KL + c];
   }
   if (lane == 0 && warp < nh) {
-    mine[(size_t)warp * p.parts * rec + R] = m;
-    mine[(size_t)warp * p.parts * rec + R + 1] = l;
+    mine[warp * head + p.rec - 4] = m;
+    mine[warp * head + p.rec - 3] = l;
   }
-  __threadfence();
-  __syncthreads();
-  uint32_t* tk = &p.tickets[i * gridDim.y + blockIdx.y];
-  if (tid == 0) ticket = atomicAdd(tk, 1u);
-  __syncthreads();
-  if (ticket != s.n_parts - 1) return;
-  __threadfence();
-  latent_merge<E>(p, i, h0, nh, s.n_parts, coef);
-  if (tid == 0) *tk = 0;
 }
 
 // ------------------------------------------------- sixteen heads as an mma tile (bf16) ----
-// Eight warps. Scores: warp w takes 16 of a tile's 64 keys and one half of the columns; the halves
-// meet in shared memory, where sixteen threads per head form the weights with a running
-// maximum. Weights x values: warp w owns every eighth slab of the value columns, NVT tiles of 8.
-constexpr int LG_THREADS = 256, LG_KEYS = 64, LG_SP = LG_KEYS + 4, LG_PS = LG_KEYS + 8;
+// Warp 8 brings the cache rows by tensor map, tiles of 32 keys in panels of 64 columns (128-byte
+// swizzle), into a ring of stages. Warps 0-7: for the scores a warp takes 16 of a tile's keys and
+// one quarter of the columns; the quarters meet in shared memory, where sixteen threads per head
+// form the weights with a running maximum; for weights x values a warp owns every eighth slab of
+// the value columns, NVT tiles of 8.
+constexpr int LG_WORKERS = 256, LG_THREADS = 288, LG_KEYS = 32, LG_SP = LG_KEYS + 4,
+              LG_PS = LG_KEYS + 8;
+constexpr int LG_PANEL = LG_KEYS * 128;  // bytes
+constexpr int LG_MAX_STAGES = 6;
+
+__device__ __forceinline__ void lg_sync() {
+  asm volatile("bar.sync 1, %0;" ::"n"(LG_WORKERS) : "memory");
+}
+// Row r, 16-byte chunk c (8 columns) of a staged tile.
+__device__ __forceinline__ uint32_t lg_addr(uint32_t tile, int r, int c) {
+  return tile + (uint32_t)((c >> 3) * LG_PANEL + r * 128 + (((c & 7) ^ (r & 7)) << 4));
+}
 
 template <int NVT>
-__global__ void __launch_bounds__(LG_THREADS) latent_group_kernel(const LatentRowsArgs p) {
-  extern __shared__ __align__(16) uint8_t sm_raw[];
-  __shared__ float corr[16], den[16], top_s[16], coef[32];
-  __shared__ uint32_t ticket;
+__global__ void __launch_bounds__(LG_THREADS)
+    latent_group_kernel(const __grid_constant__ CUtensorMap map, const LatentRowsArgs p) {
+  extern __shared__ uint8_t raw[];
+  __shared__ uint64_t full[LG_MAX_STAGES], empty[LG_MAX_STAGES];
+  __shared__ float corr[16];
+  __shared__ volatile int producer_failed, failed;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int part = blockIdx.x, h0 = blockIdx.y * 16;
   const int64_t i = blockIdx.z;
   const KvDenseLayer& kv = p.kv;
-  const int H = p.a.heads, R = p.a.rank, RD = p.a.rot, D = R + RD, KL = kv.k_ld, BS = kv.block_size;
+  const int H = p.a.heads, R = p.a.rank, RD = p.a.rot, D = R + RD, BS = kv.block_size;
   const int nh = min(16, H - h0);
-  const int dp = (D + 15) & ~15, ks = dp + 8;
-  bf16* Qs = reinterpret_cast<bf16*>(sm_raw);             // [16][ks]
-  bf16* Ks = Qs + 16 * ks;                                // two tiles [64][ks]
-  float* Sp = reinterpret_cast<float*>(Ks + 2 * LG_KEYS * ks);  // [2][16][LG_SP]
-  bf16* Ps = reinterpret_cast<bf16*>(Sp + 2 * 16 * LG_SP);      // [16][LG_PS]
-  float2* turn = reinterpret_cast<float2*>(Ps + 16 * LG_PS);    // [RD / 2]
+  const int dp = (D + 15) & ~15, ks = dp + 8, panels = (D + 63) / 64;
+  const uint32_t stage_bytes = (uint32_t)panels * LG_PANEL;
+  uint8_t* ring = raw + ((1024u - (smem_u32(raw) & 1023u)) & 1023u);
+  bf16* Qs = reinterpret_cast<bf16*>(ring + (size_t)p.stages * stage_bytes);  // [16][ks]
+  float* Sp = reinterpret_cast<float*>(Qs + 16 * ks);                         // [4][16][LG_SP]
+  bf16* Ps = reinterpret_cast<bf16*>(Sp + 4 * 16 * LG_SP);                    // [16][LG_PS]
+  float2* turn = reinterpret_cast<float2*>(Ps + 16 * LG_PS);                  // [RD / 2]
 
   pdl_launch_dependents();
   const LatentSpan s = latent_span(p, i, part);
   if ((uint32_t)part >= s.n_parts) return;
-  const bf16* pool = reinterpret_cast<const bf16*>(kv.base);
-  const int kc = dp / 8, kl = KL / 8;
-  // 16-byte pieces of a tile: thread tid takes piece (tid % 4) + 4 * n of row tid / 4
-  auto fetch = [&](uint32_t k0, int buf) {
-    const int r = tid >> 2;
-    const uint32_t j = k0 + r;
-    bool in = j < s.k_end;
-    size_t at = 0;
-    if (in) {
-      const uint32_t block = s.table[j / BS];
-      if (block < kv.num_blocks) {
-        at = kv.k_elem(block, 0, j % BS);
-      } else {
-        atomicOr(p.status, DEV_BAD_INDEX);
-        in = false;
-      }
+  const int n_tiles = (int)((s.k_end - s.k_begin + LG_KEYS - 1) / LG_KEYS);
+  if (tid == 0) {
+    for (int k = 0; k < p.stages; ++k) {
+      mbar_init(&full[k], 1);
+      mbar_init(&empty[k], LG_WORKERS / 32);
     }
-    bf16* dst = Ks + (size_t)(buf * LG_KEYS + r) * ks;
-    for (int c = tid & 3; c < kc; c += 4) {
-      const bool ok = in && c < kl;
-      cp_async16(dst + c * 8, ok ? pool + at + c * 8 : pool, ok);
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  // the first tile may be asked for before the wait when the step's own row is not in it
-  const bool early = p.r.early && s.k_begin + LG_KEYS <= s.pos;
-  if (early) fetch(s.k_begin, 0);
-  for (int k = tid; k < RD / 2; k += LG_THREADS) rope_sincos(s.pos, p.a.freq[k], &turn[k].x, &turn[k].y);
-  for (int k = tid; k < 16 * ks / 8; k += LG_THREADS)
-    reinterpret_cast<uint4*>(Qs)[k] = make_uint4(0u, 0u, 0u, 0u);
+    mbar_fence_init();
+    producer_failed = failed = 0;
+  }
   __syncthreads();
+
+  if (warp == 8) {
+    // boxes of at most a page; lane l brings piece l of a tile
+    const int box = min(BS, LG_KEYS), pieces = LG_KEYS / box;
+    const uint32_t last = (s.k_end - 1) / BS;
+    auto page_of = [&](int k) {
+      const uint32_t j = s.k_begin + (uint32_t)k * LG_KEYS + (uint32_t)min(lane, pieces - 1) * box;
+      // pages past the last key hold none that is seen: the last one stands in for them
+      uint32_t b = s.table[min(j / BS, last)];
+      if (b >= kv.num_blocks) {
+        atomicOr(p.status, DEV_BAD_INDEX);
+        b = 0;
+      }
+      return b;
+    };
+    bool waited = false;
+    int issued = 0;
+    uint32_t block = page_of(0);
+    for (int k = 0; k < n_tiles; ++k) {
+      const int st = k % p.stages;
+      const uint32_t next = k + 1 < n_tiles ? page_of(k + 1) : 0u;
+      // rows that earlier steps have stored may be asked for before the wait
+      if (!waited && !(p.r.early && s.k_begin + (uint32_t)(k + 1) * LG_KEYS <= s.pos)) {
+        pdl_wait();
+        asm volatile("fence.proxy.async;" ::: "memory");
+        waited = true;
+      }
+      const bool ok =
+          mbar_wait_bounded(&empty[st], ((uint32_t)(k / p.stages) & 1u) ^ 1u) && !failed;
+      if (!__all_sync(0xFFFFFFFFu, ok)) {
+        producer_failed = 1;
+        break;
+      }
+      if (lane == 0) mbar_arrive_expect_tx(&full[st], stage_bytes);
+      __syncwarp();
+      const int row = (int)((s.k_begin + (uint32_t)k * LG_KEYS) % BS);  // not 0: a page of 64 and more
+      if (lane < pieces)
+        for (int c = 0; c < panels; ++c)
+          tma_load_3d(ring + (size_t)st * stage_bytes + (size_t)c * LG_PANEL + lane * box * 128,
+                      &map, c * 64, row, (int)block, &full[st]);
+      issued = k + 1;
+      block = next;
+    }
+    // leave only when every copy has landed (bounded)
+    if (lane == 0)
+      for (int k = max(0, issued - p.stages); k < issued; ++k)
+        mbar_wait_bounded(&full[k % p.stages], (uint32_t)(k / p.stages) & 1u);
+    return;
+  }
+
+  for (int k = tid; k < RD / 2; k += LG_WORKERS)
+    rope_sincos(s.pos, p.a.freq[k], &turn[k].x, &turn[k].y);
+  for (int k = tid; k < 16 * ks / 8; k += LG_WORKERS)
+    reinterpret_cast<uint4*>(Qs)[k] = make_uint4(0u, 0u, 0u, 0u);
+  lg_sync();
   pdl_wait();
-  if (!early) fetch(s.k_begin, 0);
   {
     const float* ql = p.r.q_lat + i * p.r.q_row + (int64_t)h0 * p.r.q_head;
     if (R % 4 == 0 && p.r.q_head % 4 == 0 && p.r.q_row % 4 == 0) {
       const int r4 = R / 4;
-#pragma unroll 4
-      for (int k = tid; k < nh * r4; k += LG_THREADS) {
+#pragma unroll 8
+      for (int k = tid; k < nh * r4; k += LG_WORKERS) {
         const int h = k / r4, d = (k - h * r4) * 4;
         const float4 v = *reinterpret_cast<const float4*>(ql + h * p.r.q_head + d);
         *reinterpret_cast<uint2*>(Qs + h * ks + d) =
             make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
       }
     } else {
-      for (int k = tid; k < nh * R; k += LG_THREADS) {
+      for (int k = tid; k < nh * R; k += LG_WORKERS) {
         const int h = k / R, d = k - h * R;
         Qs[h * ks + d] = to_elem<bf16>(ql[h * p.r.q_head + d]);
       }
     }
     const int r2 = RD / 2;
-    for (int k = tid; k < nh * r2; k += LG_THREADS) {
+    for (int k = tid; k < nh * r2; k += LG_WORKERS) {
       const int h = k / r2, e = k - h * r2;
       const int64_t at =
           s.t * p.r.q.ld + (int64_t)(h0 + h) * (p.a.dim + RD) + p.a.dim + 2 * e;
@@ -310,6 +368,7 @@ __global__ void __launch_bounds__(LG_THREADS) latent_group_kernel(const LatentRo
       Qs[h * ks + R + 2 * e + 1] = to_elem<bf16>(y * sc.y + x * sc.x);
     }
   }
+  lg_sync();
 
   float o[NVT][4];
 #pragma unroll
@@ -318,71 +377,67 @@ __global__ void __launch_bounds__(LG_THREADS) latent_group_kernel(const LatentRo
   const float k1 = p.a.scale * L2E;
   float m = -INFINITY, l = 0.f;  // in units of log2; sixteen threads per head, l their own keys'
   const int head = tid >> 4, sub = tid & 15;
-  const int nk = dp / 16, half = warp >> 2, kb = half ? (nk + 1) / 2 : 0,
-            ke = half ? nk : (nk + 1) / 2;
+  const int nk = dp / 16, quarter = warp >> 1, kb = quarter * nk / 4, ke = (quarter + 1) * nk / 4;
   const int row = lane >> 2;
   const int v0 = warp * NVT * 8;  // first value column of the warp
   const int v_end = (R + 15) & ~15;
   const uint32_t qa = smem_u32(Qs) + (uint32_t)((lane & 15) * ks + (lane >> 4) * 8) * 2;
   const uint32_t pa = smem_u32(Ps) + (uint32_t)((lane & 15) * LG_PS + (lane >> 4) * 8) * 2;
-  int buf = 0;
-  for (uint32_t k0 = s.k_begin; k0 < s.k_end; k0 += LG_KEYS, buf ^= 1) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();  // this tile has landed, nobody reads the other buffer
-    if (k0 + LG_KEYS < s.k_end) fetch(k0 + LG_KEYS, buf ^ 1);
-    const bf16* Kt = Ks + (size_t)buf * LG_KEYS * ks;
+  const int kr = (warp & 1) * 16 + (lane & 7) + ((lane >> 4) << 3);  // key row of the lane's address
+  for (int k = 0; k < n_tiles; ++k) {
+    const int st = k % p.stages;
+    const uint32_t k0 = s.k_begin + (uint32_t)k * LG_KEYS;
+    bool ok = false;
+    for (uint32_t n = 0; n < (1u << 22) && !ok; ++n) {
+      ok = mbar_try_wait(&full[st], (uint32_t)(k / p.stages) & 1u);
+      if (!ok && (n & 63u) == 63u && producer_failed) break;
+    }
+    if (!ok) failed = 1;  // read by all after the next barrier, written by none until then
+    const uint32_t tile = smem_u32(ring) + (uint32_t)st * stage_bytes;
     {
       float c[2][4] = {};
-      const uint32_t ka = smem_u32(Kt) +
-                          (uint32_t)(((warp & 3) * 16 + (lane & 7) + ((lane >> 4) << 3)) * ks +
-                                     ((lane >> 3) & 1) * 8) * 2;
 #pragma unroll 4
       for (int kk = kb; kk < ke; ++kk) {
         uint32_t a[4], b[4];
         ldm_x4(a, qa + kk * 32);
-        ldm_x4(b, ka + kk * 32);
+        ldm_x4(b, lg_addr(tile, kr, kk * 2 + ((lane >> 3) & 1)));
         mma_bf16(c[0], a, b[0], b[1]);
         mma_bf16(c[1], a, b[2], b[3]);
       }
-      float* dst = Sp + (half * 16 + row) * LG_SP + (warp & 3) * 16 + (lane & 3) * 2;
+      float* dst = Sp + (quarter * 16 + row) * LG_SP + (warp & 1) * 16 + (lane & 3) * 2;
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt) {
         *reinterpret_cast<float2*>(dst + nt * 8) = make_float2(c[nt][0], c[nt][1]);
         *reinterpret_cast<float2*>(dst + 8 * LG_SP + nt * 8) = make_float2(c[nt][2], c[nt][3]);
       }
     }
-    __syncthreads();
+    lg_sync();
+    if (failed) break;
     {
-      const float4 x = *reinterpret_cast<const float4*>(Sp + head * LG_SP + sub * 4);
-      const float4 y = *reinterpret_cast<const float4*>(Sp + (16 + head) * LG_SP + sub * 4);
-      float v[4] = {(x.x + y.x) * k1, (x.y + y.y) * k1, (x.z + y.z) * k1, (x.w + y.w) * k1};
-      float top = -INFINITY;
+      float v[2] = {0.f, 0.f};
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        if (k0 + sub * 4 + e >= s.k_end) v[e] = -INFINITY;
-        top = fmaxf(top, v[e]);
+      for (int q = 0; q < 4; ++q) {
+        const float2 x = *reinterpret_cast<const float2*>(Sp + (q * 16 + head) * LG_SP + sub * 2);
+        v[0] += x.x, v[1] += x.y;
       }
+      v[0] = k0 + sub * 2 < s.k_end ? v[0] * k1 : -INFINITY;
+      v[1] = k0 + sub * 2 + 1 < s.k_end ? v[1] * k1 : -INFINITY;
+      float top = fmaxf(v[0], v[1]);
 #pragma unroll
       for (int q = 8; q; q >>= 1) top = fmaxf(top, __shfl_xor_sync(0xFFFFFFFFu, top, q));
       top = fmaxf(top, m);
       const float c = ex2_approx(m - top);
       m = top;
-      l *= c;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        v[e] = ex2_approx(v[e] - top);
-        l += v[e];
-      }
-      *reinterpret_cast<uint2*>(Ps + head * LG_PS + sub * 4) =
-          make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+      v[0] = ex2_approx(v[0] - top), v[1] = ex2_approx(v[1] - top);
+      l = l * c + v[0] + v[1];
+      *reinterpret_cast<uint32_t*>(Ps + head * LG_PS + sub * 2) = pack_bf16(v[0], v[1]);
       if (sub == 0) corr[head] = c;
     }
-    __syncthreads();
+    lg_sync();
     const float c0 = corr[row], c1 = corr[row + 8];
-    uint32_t a[4][4];
-#pragma unroll
-    for (int kk = 0; kk < 4; ++kk) ldm_x4(a[kk], pa + kk * 32);
-    const uint32_t va = smem_u32(Kt) + (uint32_t)((lane & 15) * ks + (lane >> 4) * 8 + v0) * 2;
+    uint32_t a[2][4];
+    ldm_x4(a[0], pa);
+    ldm_x4(a[1], pa + 32);
 #pragma unroll
     for (int nt = 0; nt < NVT; nt += 2) {
       if (v0 + nt * 8 < v_end) {
@@ -392,80 +447,76 @@ __global__ void __launch_bounds__(LG_THREADS) latent_group_kernel(const LatentRo
           o[nt + e][2] *= c1, o[nt + e][3] *= c1;
         }
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk) {
+        for (int kk = 0; kk < 2; ++kk) {
           uint32_t b[4];
-          ldm_x4_t(b, va + (uint32_t)(kk * 16 * ks + nt * 8) * 2);
+          ldm_x4_t(b, lg_addr(tile, kk * 16 + (lane & 15), v0 / 8 + nt + (lane >> 4)));
           mma_bf16(o[nt], a[kk], b[0], b[1]);
           mma_bf16(o[nt + 1], a[kk], b[2], b[3]);
         }
       }
     }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[st]);
   }
 #pragma unroll
   for (int q = 8; q; q >>= 1) l += __shfl_xor_sync(0xFFFFFFFFu, l, q);
-  __syncthreads();  // corr has been read
-  if (sub == 0) {
-    top_s[head] = m * (1.0f / L2E);
-    den[head] = l;
-    if (head < nh) {
+  if (failed) {
+    if (tid == 0) atomicOr(p.status, DEV_WAIT_TIMEOUT);
+    return;
+  }
+  if (p.parts == 1) {
+    lg_sync();  // corr has been read
+    if (sub == 0 && head < nh) {
       const float sink = p.a.sink[h0 + head] * L2E, top = fmaxf(m, sink), c = exp2f(m - top);
       corr[head] = c / (l * c + exp2f(sink - top));
     }
-  }
-  __syncthreads();
-  if (s.n_parts == 1) {
+    lg_sync();
 #pragma unroll
     for (int nt = 0; nt < NVT; ++nt)
 #pragma unroll
-      for (int e = 0; e < 4; e += 2) {
-        const int h = row + (e >> 1) * 8, c = v0 + nt * 8 + (lane & 3) * 2;
-        if (h >= nh || c >= R) continue;
-        const int64_t at = i * p.r.out_row + (h0 + h) * p.r.out_head + c;
-        const float x = o[nt][e] * corr[h], y = o[nt][e + 1] * corr[h];
-        if (p.r.out_f32) {
-          float* dst = static_cast<float*>(p.r.out) + at;
-          dst[0] = x;
-          if (c + 1 < R) dst[1] = y;
-        } else {
-          bf16* dst = static_cast<bf16*>(p.r.out) + at;
-          dst[0] = to_elem<bf16>(x);
-          if (c + 1 < R) dst[1] = to_elem<bf16>(y);
-        }
+      for (int e = 0; e < 4; ++e) {
+        const int h = row + (e >> 1) * 8, c = v0 + nt * 8 + (lane & 3) * 2 + (e & 1);
+        if (h < nh && c < R) latent_out<bf16>(p, i, h0 + h, c, o[nt][e] * corr[h]);
       }
     return;
   }
-  const size_t rec = (size_t)R + 2;
-  float* mine = p.partial + ((size_t)i * H + h0) * p.parts * rec + part * rec;
+  float* mine = p.partial + (((size_t)i * H + h0) * p.parts + part) * p.rec;
+  const size_t step = (size_t)p.parts * p.rec;
 #pragma unroll
   for (int nt = 0; nt < NVT; ++nt)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int h = row + (e >> 1) * 8, c = v0 + nt * 8 + (lane & 3) * 2 + (e & 1);
-      if (h < nh && c < R) mine[(size_t)h * p.parts * rec + c] = o[nt][e];
+    for (int e = 0; e < 4; e += 2) {
+      const int h = row + (e >> 1) * 8, c = v0 + nt * 8 + (lane & 3) * 2;
+      // an odd last column takes the place of the pad behind it along
+      if (h < nh && c < R)
+        *reinterpret_cast<float2*>(mine + h * step + c) = make_float2(o[nt][e], o[nt][e + 1]);
     }
-  if (tid < nh) {
-    mine[(size_t)tid * p.parts * rec + R] = top_s[tid];
-    mine[(size_t)tid * p.parts * rec + R + 1] = den[tid];
+  if (sub == 0 && head < nh) {
+    mine[head * step + p.rec - 4] = m * (1.0f / L2E);
+    mine[head * step + p.rec - 3] = l;
   }
-  __threadfence();
-  __syncthreads();
-  uint32_t* tk = &p.tickets[i * gridDim.y + blockIdx.y];
-  if (tid == 0) ticket = atomicAdd(tk, 1u);
-  __syncthreads();
-  if (ticket != s.n_parts - 1) return;
-  __threadfence();
-  latent_merge<bf16>(p, i, h0, nh, s.n_parts, coef);
-  if (tid == 0) *tk = 0;
 }
 
 template <int NVT>
-static int32_t group_launch(kanso_cuda_ctx* ctx, dim3 grid, size_t smem, const LatentRowsArgs& p) {
+static int32_t group_launch(kanso_cuda_ctx* ctx, dim3 grid, size_t smem, const CUtensorMap& map,
+                            const LatentRowsArgs& p) {
   int32_t st = allow_max_smem(ctx, (const void*)latent_group_kernel<NVT>);
   if (st) return st;
   const cudaError_t e =
-      launch_dependent(ctx, latent_group_kernel<NVT>, grid, dim3(LG_THREADS), smem, p);
+      launch_dependent(ctx, latent_group_kernel<NVT>, grid, dim3(LG_THREADS), smem, map, p);
   if (e != cudaSuccess) return cuda_fail(ctx, e, "latent attention launch");
   return after_launch(ctx, "latent_group");
+}
+
+// Stages of the tile form's ring and its shared memory; 0 stages: it does not fit.
+static int group_stages(const LatentAttn& a, uint32_t k_dim, size_t* smem) {
+  const size_t stage = (size_t)((k_dim + 63) / 64) * LG_PANEL;
+  const size_t rest = 1024 + (size_t)16 * (((k_dim + 15u) & ~15u) + 8) * 2 + 4 * 16 * LG_SP * 4 +
+                      16 * LG_PS * 2 + (size_t)a.rot * 4;
+  int n = LG_MAX_STAGES;
+  while (n > 0 && n * stage + rest > 222 * 1024) --n;
+  *smem = n * stage + rest;
+  return n >= 2 ? n : 0;
 }
 
 int32_t launch_latent_attn_rows(kanso_cuda_ctx* ctx, int32_t compute, const LatentAttn& a,
@@ -474,69 +525,85 @@ int32_t launch_latent_attn_rows(kanso_cuda_ctx* ctx, int32_t compute, const Late
   *handled = true;
   if (r.n > 65535)
     return fail(ctx, KANSO_ERR_UNSUPPORTED, "attention: %lld rows in one launch", (long long)r.n);
-  const int dp = (int)((kv.k_dim + 15u) & ~15u), ks = dp + 8;
-  const size_t gsmem = ((size_t)16 * ks + 2 * (size_t)LG_KEYS * ks) * 2 + 2 * 16 * LG_SP * 4 +
-                       16 * LG_PS * 2 + (size_t)a.rot * 4;
-  const bool fits = compute == KANSO_COMPUTE_BF16 && a.rank <= 1024 && gsmem <= 224 * 1024;
-  if (path == 2 && !fits) {
-    *handled = false;
-    return KANSO_OK;
-  }
-  const bool group = fits && path != 1;
   LatentRowsArgs p;
   p.a = a;
   p.kv = kv;
   p.r = r;
   p.partial = nullptr;
-  p.tickets = ctx->pa_tickets;
-  p.tile = group ? LG_KEYS : LR_TILE;
   p.status = ctx->dev_status;
+  size_t smem = 0;
+  p.stages = group_stages(a, kv.k_dim, &smem);
+  const uint32_t bs = kv.block_size;
+  bool group = path != 1 && compute == KANSO_COMPUTE_BF16 && a.rank <= 1024 && p.stages &&
+               (bs == 8 || bs == 16 || bs % 32 == 0) && kv.num_blocks < (1u << 31);
+  CUtensorMap map;
+  if (group) {
+    TmEncodeFn encode = tm_encoder();
+    group = encode && tm_map3(encode, kv.base, kv.k_ld, bs, kv.num_blocks, kv.k_ld, kv.rec_elems,
+                              std::min<uint32_t>(bs, LG_KEYS), 1, &map);
+  }
+  if (path == 2 && !group) {
+    *handled = false;
+    return KANSO_OK;
+  }
+  p.tile = group ? LG_KEYS : LR_TILE;
+  p.rec = ((a.rank + 3u) & ~3u) + 4;
   const uint32_t HB = group ? (a.heads + 15) / 16 : (a.heads + LR_HEADS - 1) / LR_HEADS;
   const uint32_t tiles = std::max(1u, (r.max_keys + p.tile - 1) / p.tile);
   const uint64_t ctas = (uint64_t)r.n * HB;
+  // Shares of the keys. The tile form: the split with the shortest run of waves, a wave being a
+  // share's tiles and a few tiles' worth of fixed work; the plain form: four CTAs per SM.
   uint32_t parts = 1;
-  if (ctas <= kanso_cuda_ctx::kPaTickets) {
-    if (group) {
-      // the split with the shortest run of waves, a wave being a share's tiles and about two tiles'
-      // worth of fixed work
-      const uint64_t per_sm = std::max<uint64_t>(
-          1, std::min<uint64_t>(4, (uint64_t)ctx->smem_per_sm / (gsmem + 2048)));
-      const uint64_t resident = (uint64_t)ctx->sm_count * per_sm;
-      uint64_t best = ~0ull;
-      for (uint32_t n = 1; n <= tiles; ++n) {
-        const uint64_t cost = (ctas * n + resident - 1) / resident * ((tiles + n - 1) / n + 2);
-        if (cost < best) {
-          best = cost;
-          parts = n;
-        }
+  if (group) {
+    const uint64_t per_sm = std::max<uint64_t>(
+        1, std::min<uint64_t>(4, (uint64_t)ctx->smem_per_sm / (smem + 1200)));
+    const uint64_t resident = (uint64_t)ctx->sm_count * per_sm;
+    uint64_t best = ~0ull;
+    for (uint32_t n = 1; n <= std::min(tiles, 256u); ++n) {
+      const uint64_t cost =
+          (ctas * n + resident - 1) / resident * ((tiles + n - 1) / n + 6) + (n > 1 ? 6 : 0);
+      if (cost < best) {
+        best = cost;
+        parts = n;
       }
-    } else {
-      parts = (uint32_t)std::min<uint64_t>(
-          tiles, std::max<uint64_t>(1, 4ull * ctx->sm_count / ctas));
     }
+  } else {
+    parts = (uint32_t)std::min<uint64_t>(std::min(tiles, 256u),
+                                         std::max<uint64_t>(1, 4ull * ctx->sm_count / ctas));
   }
   const uint32_t per = (tiles + parts - 1) / parts;
   p.parts = (tiles + per - 1) / per;
   if (p.parts > 1) {
-    p.partial = (float*)ctx_scratch(ctx, (size_t)r.n * a.heads * p.parts * (a.rank + 2) * 4);
+    p.partial = (float*)ctx_scratch(ctx, (size_t)r.n * a.heads * p.parts * p.rec * 4);
     if (!p.partial) return KANSO_ERR_DEVICE;
   }
   const dim3 grid(p.parts, HB, (unsigned)r.n);
+  int32_t st;
   if (group) {
-    if (a.rank <= 128) return group_launch<2>(ctx, grid, gsmem, p);
-    if (a.rank <= 256) return group_launch<4>(ctx, grid, gsmem, p);
-    if (a.rank <= 512) return group_launch<8>(ctx, grid, gsmem, p);
-    return group_launch<16>(ctx, grid, gsmem, p);
+    st = a.rank <= 128   ? group_launch<2>(ctx, grid, smem, map, p)
+         : a.rank <= 256 ? group_launch<4>(ctx, grid, smem, map, p)
+         : a.rank <= 512 ? group_launch<8>(ctx, grid, smem, map, p)
+                         : group_launch<16>(ctx, grid, smem, map, p);
+    if (st) return st;
+  } else {
+    smem = (size_t)2 * LR_HEADS * kv.k_ld * 4;
+    if (smem > 200 * 1024)
+      return fail(ctx, KANSO_ERR_UNSUPPORTED, "latent attention: cache rows of %u columns",
+                  kv.k_dim);
+    auto kern =
+        compute == KANSO_COMPUTE_BF16 ? latent_rows_kernel<bf16> : latent_rows_kernel<float>;
+    if ((st = allow_max_smem(ctx, (const void*)kern))) return st;
+    const cudaError_t e = launch_dependent(ctx, kern, grid, dim3(LR_THREADS), smem, p);
+    if (e != cudaSuccess) return cuda_fail(ctx, e, "latent attention launch");
+    if ((st = after_launch(ctx, "latent_rows"))) return st;
   }
-  const size_t smem = (size_t)2 * LR_HEADS * kv.k_ld * 4;
-  if (smem > 200 * 1024)
-    return fail(ctx, KANSO_ERR_UNSUPPORTED, "latent attention: cache rows of %u columns", kv.k_dim);
-  auto kern = compute == KANSO_COMPUTE_BF16 ? latent_rows_kernel<bf16> : latent_rows_kernel<float>;
-  int32_t st = allow_max_smem(ctx, (const void*)kern);
-  if (st) return st;
-  const cudaError_t e = launch_dependent(ctx, kern, grid, dim3(LR_THREADS), smem, p);
-  if (e != cudaSuccess) return cuda_fail(ctx, e, "latent attention launch");
-  return after_launch(ctx, "latent_rows");
+  if (p.parts == 1) return KANSO_OK;
+  auto merge =
+      compute == KANSO_COMPUTE_BF16 ? latent_merge_kernel<bf16> : latent_merge_kernel<float>;
+  const cudaError_t e = launch_dependent(ctx, merge, dim3(a.heads, (unsigned)r.n),
+                                         dim3(LM_THREADS), (size_t)p.parts * 4, p);
+  if (e != cudaSuccess) return cuda_fail(ctx, e, "latent merge launch");
+  return after_launch(ctx, "latent_merge");
 }
 
 }  // namespace kanso

@@ -677,7 +677,7 @@ int32_t MiguraxModel::memory_tiles(kanso_cuda_kv* kv, size_t l, const DenseStep&
   if (chunks) {
     MlstmArgs b = a;
     b.portions = s.portions + s.n_short;
-    if ((st = launch_mlstm_chunks(ctx, b, s.n_long, chunk_mem, s.T))) return st;
+    if ((st = launch_mlstm_chunks(ctx, b, s.n_long, s.max_long_rows, chunk_mem, s.T))) return st;
   }
   return launch_head_norm_gate(ctx, compute, a, ly.head_norm, cfg.eps, ao, ly.o.ld, s.T);
 }

@@ -220,7 +220,7 @@ int32_t kanso_cuda_mlstm(kanso_cuda_ctx* ctx, kanso_cuda_kv* kv, uint32_t layer,
                      : fail(ctx, KANSO_ERR_UNSUPPORTED, "mlstm: heads of %u columns", a.dim);
   const size_t bytes = mlstm_chunk_bytes(a.heads, a.dim, a.vdim, p->num_rows);
   if ((st = mem.copy(nullptr, bytes, &work))) return st;
-  return launch_mlstm_chunks(ctx, a, 1, work, p->num_rows);
+  return launch_mlstm_chunks(ctx, a, 1, p->num_rows, work, p->num_rows);
 }
 
 int32_t kanso_cuda_head_norm_gate(kanso_cuda_ctx* ctx, const float* o, const float* y,

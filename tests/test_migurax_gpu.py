@@ -177,6 +177,7 @@ class LatentCase:
     (33, 264, 6, 32, 333, 0.05, 50.0),
     (5, 512, 64, 16, 700, 0.04, 10000.0),
     (3, 640, 16, 16, 129, 0.03, 3.0),
+    (4, 40, 24, 64, 500, 0.1, 700.0),
 ])
 def test_latent_attention(kb, ctx, torch_cuda, compute, path, H, rank, rot, bs, n, scale, base):
     torch = torch_cuda
@@ -184,6 +185,11 @@ def test_latent_attention(kb, ctx, torch_cuda, compute, path, H, rank, rot, bs, 
     case = LatentCase(kb, ctx, torch, rng, rng.standard_normal((n, rank + rot)) * 2,
                       rng.uniform(0.5, 1.5, rank), rank, base, bs, compute)
     sink = rng.uniform(-3, 6, H)
+    if path == 2 and bs == 5:  # pages that do not make up a tile
+        with pytest.raises(kb.KansoError) as e:
+            case.attend(np.zeros((1, H, rank)), np.zeros((1, H, 7 + rot)), [n - 1], scale, sink, path)
+        assert e.value.code == kb.ERR_UNSUPPORTED
+        return
     for rows in (np.arange(n), [n - 1], [0, 1, n // 2], np.arange(60, 70) % n):
         rows = np.asarray(rows)
         q_lat = rng.standard_normal((len(rows), H, rank)) * 3
