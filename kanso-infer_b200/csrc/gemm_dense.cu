@@ -17,6 +17,7 @@
 //
 // f32: 64 x 64 tiles on the FMA units.
 #include <algorithm>
+#include <type_traits>
 
 #include "dense.cuh"
 #include "tc05.cuh"
@@ -114,7 +115,37 @@ struct GdShape {
   static constexpr size_t kSmem = (size_t)kStage * kStages + 1024;
 };
 
-template <int NT, bool DUAL, bool ACT>
+// The results of column n (and n + 128) through bias and activation to their places.
+template <int NT, bool DUAL, typename O>
+__device__ __forceinline__ void ext_rows(const GemmDenseArgs& a, const RowPlace& place, O* out,
+                                         uint32_t tmem, int n, int64_t first, int valid) {
+  const float b0 = a.bias_of(n), b1 = DUAL ? a.bias_of(n + 128) : 0.f;
+  const bool in0 = n < a.n_end, in1 = DUAL && n + 128 < a.n_end, sq = a.relu2;
+  const float low = sq ? 0.f : -INFINITY;
+  const int64_t ld = a.out_ld;
+  out += place.shift + n;
+  for (int c = 0; c < NT; c += 16) {
+    if (c >= valid) break;
+    uint32_t r0[16], r1[16];
+    tmem_ld16(tmem + c, r0);
+    if (DUAL) tmem_ld16(tmem + NT + c, r1);
+    O* o = out + (first + c) * ld;
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      if (c + j >= valid) continue;
+      const float x = fmaxf(__uint_as_float(r0[j]) + b0, low);
+      O* at = place.list ? out + place.list[first + c + j - place.first] * ld : o + j * ld;
+      if (in0) at[0] = to_elem<O>(sq ? x * x : x);
+      if (DUAL) {
+        const float y = fmaxf(__uint_as_float(r1[j]) + b1, low);
+        if (in1) at[128] = to_elem<O>(sq ? y * y : y);
+      }
+    }
+  }
+}
+
+// EXT: results go through bias, activation, element type or place (GemmOut).
+template <int NT, bool DUAL, bool ACT, bool EXT>
 __global__ void __launch_bounds__(GD_THREADS)
     gemm_dense_kernel(const __grid_constant__ CUtensorMap wmap,
                       const __grid_constant__ CUtensorMap wmap2,
@@ -225,44 +256,34 @@ __global__ void __launch_bounds__(GD_THREADS)
     const int n = n0 + warp * 32 + lane;  // a warp reaches its own quarter of the TMEM lanes
     const uint32_t lane_base = tmem + ((uint32_t)(warp * 32) << 16);
     const int valid = (int)min((int64_t)NT, tile_end - tile_first);
-    const RowPlace place(a, tile_group);
-    const float b0 = a.bias_of(n), b1 = DUAL ? a.bias_of(n + 128) : 0.f;
-    const bool in0 = n < a.n_end, in1 = n + 128 < a.n_end;
-    for (int c = 0; c < NT / 16; ++c) {
+    if (EXT) {
+      const RowPlace place(a, tile_group);
+      if (a.elem)
+        ext_rows<NT, DUAL>(a, place, static_cast<bf16*>(a.out), lane_base, n, tile_first, valid);
+      else
+        ext_rows<NT, DUAL>(a, place, static_cast<float*>(a.out) + (int64_t)blockIdx.z * a.part_stride,
+                           lane_base, n, tile_first, valid);
+    }
+    for (int c = 0; c < NT / 16 && !EXT; ++c) {
       if (c * 16 >= valid) break;
       uint32_t r0[16], r1[16];
       tmem_ld16(lane_base + c * 16, r0);
       if (DUAL) tmem_ld16(lane_base + NT + c * 16, r1);
-      if (ACT) {
 #pragma unroll
-        for (int j = 0; j < 16; ++j) {
-          if (c * 16 + j >= valid) continue;
+      for (int j = 0; j < 16; ++j) {
+        const int m = c * 16 + j;
+        if (m >= valid) continue;
+        const int64_t row = tile_first + m;
+        if (ACT) {
           // the pad columns multiply weight rows that were zero-filled: they come out as zero
           const float g = __uint_as_float(r0[j]), u = __uint_as_float(r1[j]);
           if (n < a.out_ld)
-            static_cast<bf16*>(a.out)[(tile_first + c * 16 + j) * a.out_ld + n] =
-                to_elem<bf16>(silu(g) * u);
-        }
-      } else if (a.elem) {
-#pragma unroll
-        for (int j = 0; j < 16; ++j) {
-          if (c * 16 + j >= valid) continue;
-          float v0 = __uint_as_float(r0[j]) + b0, v1 = DUAL ? __uint_as_float(r1[j]) + b1 : 0.f;
-          if (a.relu2) v0 = relu_squared(v0), v1 = relu_squared(v1);
-          bf16* o = static_cast<bf16*>(a.out) + place.at(tile_first + c * 16 + j, a.out_ld) + n;
-          if (in0) o[0] = to_elem<bf16>(v0);
-          if (DUAL && in1) o[128] = to_elem<bf16>(v1);
-        }
-      } else {
-        float* part = static_cast<float*>(a.out) + (int64_t)blockIdx.z * a.part_stride + n;
-#pragma unroll
-        for (int j = 0; j < 16; ++j) {
-          if (c * 16 + j >= valid) continue;
-          float v0 = __uint_as_float(r0[j]) + b0, v1 = DUAL ? __uint_as_float(r1[j]) + b1 : 0.f;
-          if (a.relu2) v0 = relu_squared(v0), v1 = relu_squared(v1);
-          float* o = part + place.at(tile_first + c * 16 + j, a.out_ld);
-          if (in0) o[0] = v0;
-          if (DUAL && in1) o[128] = v1;
+            static_cast<bf16*>(a.out)[row * a.out_ld + n] = to_elem<bf16>(silu(g) * u);
+        } else {
+          float* o = static_cast<float*>(a.out) + (int64_t)blockIdx.z * a.part_stride +
+                     row * a.out_ld;
+          if (n < a.rows) o[n] = __uint_as_float(r0[j]);
+          if (DUAL && n + 128 < a.rows) o[n + 128] = __uint_as_float(r1[j]);
         }
       }
     }
@@ -387,14 +408,14 @@ static int32_t rows_map(kanso_cuda_ctx* ctx, const void* x, int64_t T, int64_t c
   return KANSO_OK;
 }
 
-template <int NT, bool DUAL, bool ACT>
+template <int NT, bool DUAL, bool ACT, bool EXT>
 static int32_t gd_launch(kanso_cuda_ctx* ctx, dim3 grid, const CUtensorMap& wm,
                          const CUtensorMap& wm2, const CUtensorMap& xm, const GemmDenseArgs& a) {
-  int32_t st = allow_max_smem(ctx, (const void*)gemm_dense_kernel<NT, DUAL, ACT>);
+  auto kern = gemm_dense_kernel<NT, DUAL, ACT, EXT>;
+  int32_t st = allow_max_smem(ctx, (const void*)kern);
   if (st) return st;
-  const cudaError_t e = launch_dependent(ctx, gemm_dense_kernel<NT, DUAL, ACT>, grid,
-                                         dim3(GD_THREADS), GdShape<NT, DUAL, ACT>::kSmem, wm, wm2,
-                                         xm, a);
+  const cudaError_t e = launch_dependent(ctx, kern, grid, dim3(GD_THREADS),
+                                         GdShape<NT, DUAL, ACT>::kSmem, wm, wm2, xm, a);
   if (e != cudaSuccess) return cuda_fail(ctx, e, "gemm_dense launch");
   return after_launch(ctx, "gemm_dense");
 }
@@ -443,16 +464,23 @@ int32_t launch_gemm(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat& w, con
   a.steps_per_split = (a.k_steps + sp - 1) / sp;
   sp = (a.k_steps + a.steps_per_split - 1) / a.steps_per_split;
   *splits = sp;
-  if (dual) {
-    const dim3 grid((unsigned)((w.rows + 255) / 256), (unsigned)ty, (unsigned)sp);
-    return gd_launch<128, true, false>(ctx, grid, wm, wm, xm, a);
-  }
+  const bool ext = o.bias || o.relu2 || o.elem || o.group_step;
+  auto launch = [&](auto n, auto two, dim3 grid) {
+    constexpr int NT = decltype(n)::value;
+    constexpr bool DUAL = decltype(two)::value;
+    return ext ? gd_launch<NT, DUAL, false, true>(ctx, grid, wm, wm, xm, a)
+               : gd_launch<NT, DUAL, false, false>(ctx, grid, wm, wm, xm, a);
+  };
+  using std::integral_constant;
+  if (dual)
+    return launch(integral_constant<int, 128>(), std::true_type(),
+                  dim3((unsigned)((w.rows + 255) / 256), (unsigned)ty, (unsigned)sp));
   const dim3 grid((unsigned)tx, (unsigned)ty, (unsigned)sp);
   switch (nt) {
-    case 16: return gd_launch<16, false, false>(ctx, grid, wm, wm, xm, a);
-    case 32: return gd_launch<32, false, false>(ctx, grid, wm, wm, xm, a);
-    case 64: return gd_launch<64, false, false>(ctx, grid, wm, wm, xm, a);
-    default: return gd_launch<128, false, false>(ctx, grid, wm, wm, xm, a);
+    case 16: return launch(integral_constant<int, 16>(), std::false_type(), grid);
+    case 32: return launch(integral_constant<int, 32>(), std::false_type(), grid);
+    case 64: return launch(integral_constant<int, 64>(), std::false_type(), grid);
+    default: return launch(integral_constant<int, 128>(), std::false_type(), grid);
   }
 }
 
@@ -479,10 +507,10 @@ int32_t launch_gemm_gate_up(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat
   a.k_steps = a.steps_per_split = (int)((gate.cols + GD_K - 1) / GD_K);
   const dim3 grid((unsigned)((gate.rows + 127) / 128), (unsigned)tiles_of(r, nt));
   switch (nt) {
-    case 16: return gd_launch<16, true, true>(ctx, grid, gm, um, xm, a);
-    case 32: return gd_launch<32, true, true>(ctx, grid, gm, um, xm, a);
-    case 64: return gd_launch<64, true, true>(ctx, grid, gm, um, xm, a);
-    default: return gd_launch<128, true, true>(ctx, grid, gm, um, xm, a);
+    case 16: return gd_launch<16, true, true, false>(ctx, grid, gm, um, xm, a);
+    case 32: return gd_launch<32, true, true, false>(ctx, grid, gm, um, xm, a);
+    case 64: return gd_launch<64, true, true, false>(ctx, grid, gm, um, xm, a);
+    default: return gd_launch<128, true, true, false>(ctx, grid, gm, um, xm, a);
   }
 }
 
