@@ -348,12 +348,21 @@ struct LatentStore {
   RowMap map;
   int* status = nullptr;
 };
+// Sine and cosine of the thread's first pair of columns: nothing in front is needed for them.
+__device__ __forceinline__ float2 latent_turn(const LatentStore& s, int64_t t) {
+  float2 r = make_float2(0.f, 1.f);
+  if (threadIdx.x < s.a.rot / 2)
+    rope_sincos(s.map.positions[t], s.a.freq[threadIdx.x], &r.x, &r.y);
+  return r;
+}
 template <typename E>
-__device__ __forceinline__ void latent_store_row(const LatentStore& s, int64_t t, float* red) {
+__device__ __forceinline__ void latent_store_row(const LatentStore& s, int64_t t, float2 turn,
+                                                 float* red) {
   const LatentDown& p = s.down;
   const float* src = p.d + t * p.ld + p.q_rank;
   auto value = [&](int i) {
     float v = src[i];
+#pragma unroll 3
     for (int k = 1; k < p.parts; ++k) v += src[k * p.part_stride + i];
     return v;
   };
@@ -364,8 +373,15 @@ __device__ __forceinline__ void latent_store_row(const LatentStore& s, int64_t t
   const uint32_t place = pos / kv.block_size;
   uint32_t block = kv.num_blocks;
   if (place < s.map.max_blocks) block = s.map.tables[(int64_t)seq * s.map.max_blocks + place];
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < R; i += blockDim.x) {
+  constexpr int KEEP = 4;  // values a thread keeps between the two passes
+  float kept[KEEP], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    kept[k] = i < R ? value(i) : 0.f;
+    ss += kept[k] * kept[k];
+  }
+  for (int i = threadIdx.x + KEEP * blockDim.x; i < R; i += blockDim.x) {
     const float v = value(i);
     ss += v * v;
   }
@@ -376,14 +392,18 @@ __device__ __forceinline__ void latent_store_row(const LatentStore& s, int64_t t
   }
   const float inv = 1.0f / sqrtf(ss / (float)R + p.eps);
   E* dst = reinterpret_cast<E*>(kv.base) + kv.k_elem(block, 0, pos % kv.block_size);
-  for (int i = threadIdx.x; i < R; i += blockDim.x)
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    if (i < R) dst[i] = to_elem<E>(kept[k] * inv * p.c_norm[i]);
+  }
+  for (int i = threadIdx.x + KEEP * blockDim.x; i < R; i += blockDim.x)
     dst[i] = to_elem<E>(value(i) * inv * p.c_norm[i]);
   for (int i = threadIdx.x; i < RD / 2; i += blockDim.x) {
-    float sn, cs;
-    rope_sincos(pos, s.a.freq[i], &sn, &cs);
+    if (i != threadIdx.x) rope_sincos(pos, s.a.freq[i], &turn.x, &turn.y);
     const float u = value(R + 2 * i), v = value(R + 2 * i + 1);
-    dst[R + 2 * i] = to_elem<E>(u * cs - v * sn);
-    dst[R + 2 * i + 1] = to_elem<E>(v * cs + u * sn);
+    dst[R + 2 * i] = to_elem<E>(u * turn.y - v * turn.x);
+    dst[R + 2 * i + 1] = to_elem<E>(v * turn.y + u * turn.x);
   }
 }
 // The store, and the normed query latents cq [T][q_rank ld] in the products' element type.

@@ -2,6 +2,7 @@
 // x += mult * rmsnorm(y) * w, the norm of wanted rows, q / k norm with the store to the pool, and
 // the routing of rows to experts. All of it in 32-bit; what feeds a matrix product is also
 // written in the product's element type.
+#include <algorithm>
 #include <cmath>
 
 #include "dense.cuh"
@@ -357,43 +358,75 @@ __global__ void __launch_bounds__(DR_THREADS)
     latent_down_kernel(const LatentStore s, E* __restrict__ cq, int64_t cq_ld) {
   __shared__ float red[32];
   pdl_launch_dependents();
-  pdl_wait();
   const int64_t t = blockIdx.x;
   if (blockIdx.y == 1) {  // the cache row
-    latent_store_row<E>(s, t, red);
+    const float2 turn = latent_turn(s, t);
+    pdl_wait();
+    latent_store_row<E>(s, t, turn, red);
     return;
   }
+  pdl_wait();
   const LatentDown& p = s.down;
   const float* src = p.d + t * p.ld;
+  const int Q = (int)p.q_rank;
   auto value = [&](int i) {
     float v = src[i];
+#pragma unroll 3
     for (int k = 1; k < p.parts; ++k) v += src[k * p.part_stride + i];
     return v;
   };
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < (int)p.q_rank; i += DR_THREADS) {
+  constexpr int KEEP = 6;  // values a thread keeps between the two passes
+  float kept[KEEP], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = threadIdx.x + k * DR_THREADS;
+    kept[k] = i < Q ? value(i) : 0.f;
+    ss += kept[k] * kept[k];
+  }
+  for (int i = threadIdx.x + KEEP * DR_THREADS; i < Q; i += DR_THREADS) {
     const float v = value(i);
     ss += v * v;
   }
   ss = block_sum(ss, red);
-  const float inv = 1.0f / sqrtf(ss / (float)p.q_rank + p.eps);
-  for (int i = threadIdx.x; i < cq_ld; i += DR_THREADS)
-    cq[t * cq_ld + i] = to_elem<E>(i < (int)p.q_rank ? value(i) * inv * p.q_norm[i] : 0.f);
+  const float inv = 1.0f / sqrtf(ss / (float)Q + p.eps);
+  E* dst = cq + t * cq_ld;
+#pragma unroll
+  for (int k = 0; k < KEEP; ++k) {
+    const int i = threadIdx.x + k * DR_THREADS;
+    if (i < cq_ld) dst[i] = to_elem<E>(i < Q ? kept[k] * inv * p.q_norm[i] : 0.f);
+  }
+  for (int i = threadIdx.x + KEEP * DR_THREADS; i < cq_ld; i += DR_THREADS)
+    dst[i] = to_elem<E>(i < Q ? value(i) * inv * p.q_norm[i] : 0.f);
 }
 
+// blockIdx.y = a part of the heads
 template <typename E>
 __global__ void __launch_bounds__(DR_THREADS)
     latent_q_heads_kernel(const LatentAttn a, const LatentQuery q, const uint32_t* __restrict__ rows,
                           int64_t n, E* __restrict__ out, int ld) {
   pdl_launch_dependents();
-  pdl_wait();
   const int64_t i = blockIdx.x, t = rows ? rows[i] : i;
+  const int per = ((int)a.heads + gridDim.y - 1) / gridDim.y, h0 = blockIdx.y * per,
+            h1 = min(h0 + per, (int)a.heads), D = a.dim, Q = D + a.rot;
   const float* src = q.q + t * q.ld;
-  for (int k = threadIdx.x; k < (int)a.heads * ld; k += DR_THREADS) {
-    const int h = k / ld, d = k - h * ld;
+  pdl_wait();
+  if (D % 8 == 0 && Q % 4 == 0 && q.ld % 4 == 0 && q.part_stride % 4 == 0) {
+    for (int k = threadIdx.x * 4; k < (h1 - h0) * D; k += DR_THREADS * 4) {
+      const int h = h0 + k / D, d = k % D;
+      const float* at = src + (int64_t)h * Q + d;
+      float4 v = *reinterpret_cast<const float4*>(at);
+#pragma unroll 3
+      for (int p = 1; p < q.parts; ++p)
+        add4(v, *reinterpret_cast<const float4*>(at + p * q.part_stride));
+      store4(out + ((int64_t)h * n + i) * ld + d, v.x, v.y, v.z, v.w);
+    }
+    return;
+  }
+  for (int k = threadIdx.x; k < (h1 - h0) * ld; k += DR_THREADS) {
+    const int h = h0 + k / ld, d = k % ld;
     float v = 0.f;
-    if (d < (int)a.dim) {
-      const float* at = src + (int64_t)h * (a.dim + a.rot) + d;
+    if (d < D) {
+      const float* at = src + (int64_t)h * Q + d;
       v = at[0];
       for (int p = 1; p < q.parts; ++p) v += at[p * q.part_stride];
     }
@@ -646,11 +679,17 @@ int32_t launch_latent_down(kanso_cuda_ctx* ctx, int32_t compute, const LatentSto
 int32_t launch_latent_q_heads(kanso_cuda_ctx* ctx, int32_t compute, const LatentAttn& a,
                               const LatentQuery& q, const uint32_t* rows, int64_t n, void* out) {
   const int ld = (int)round_up8(a.dim);
-  if (compute == KANSO_COMPUTE_BF16)
-    DR_LAUNCH(latent_q_heads_kernel<bf16>, n, DR_THREADS, 0, "latent_q_heads", a, q, rows, n,
-              (bf16*)out, ld);
-  DR_LAUNCH(latent_q_heads_kernel<float>, n, DR_THREADS, 0, "latent_q_heads", a, q, rows, n,
-            (float*)out, ld);
+  // few rows: a thread's four columns in one go
+  const int64_t trips = ((int64_t)a.heads * ld + DR_THREADS * 4 - 1) / (DR_THREADS * 4);
+  const dim3 grid((unsigned)n, (unsigned)std::min<int64_t>({trips, (int64_t)a.heads, n > 512 ? 1 : 8}));
+  const cudaError_t e =
+      compute == KANSO_COMPUTE_BF16
+          ? launch_dependent(ctx, latent_q_heads_kernel<bf16>, grid, dim3(DR_THREADS), 0, a, q,
+                             rows, n, (bf16*)out, ld)
+          : launch_dependent(ctx, latent_q_heads_kernel<float>, grid, dim3(DR_THREADS), 0, a, q,
+                             rows, n, (float*)out, ld);
+  if (e != cudaSuccess) return cuda_fail(ctx, e, "latent_q_heads");
+  return after_launch(ctx, "latent_q_heads");
 }
 
 int32_t launch_latent_q_rows(kanso_cuda_ctx* ctx, const LatentAttn& a, const LatentQuery& q,

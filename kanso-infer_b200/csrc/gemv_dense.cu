@@ -130,24 +130,38 @@ struct GemvArgs {
   LatentStore store;
 };
 
-// Each head over its own root mean square, weight and gate (GemvSource::gate): a warp per head.
+// Each head over its own root mean square, weight and gate (GemvSource::gate): a warp per head, or
+// several where the heads are few. Every thread of the CTA must come here.
 __device__ __forceinline__ void gate_source(const GemvSource& s, const float* x, const float* gate,
-                                            int cols, int ld, float* xt) {
+                                            int cols, int ld, float* xt, float* red) {
   const int hd = cols / s.heads, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int h = warp; h < s.heads; h += GV_WARPS) {
+  int wph = 1;  // warps per head
+  while (wph * 2 * s.heads <= GV_WARPS) wph *= 2;
+  const int sub = warp % wph, step = wph * 32;
+  for (int h0 = 0; h0 < s.heads; h0 += GV_WARPS / wph) {
+    const int h = h0 + warp / wph;
+    const int first = h * hd + sub * 32 + lane, end = h < s.heads ? (h + 1) * hd : 0;
     float ss = 0.f;
-    for (int i = lane; i < hd; i += 32) {
-      const float v = x[h * hd + i];
+#pragma unroll 4
+    for (int i = first; i < end; i += step) {
+      const float v = x[i];
+      float g = gate[i];
+      for (int p = 1; p < s.parts; ++p) g += gate[p * s.part_stride + i];
+      xt[xs_index(i, ld)] = v * s.norm_w[i] / (1.0f + expf(-g));
       ss += v * v;
     }
 #pragma unroll
     for (int o = 16; o; o >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, o);
-    const float inv = 1.0f / sqrtf(ss / (float)hd + s.eps);
-    for (int i = h * hd + lane; i < (h + 1) * hd; i += 32) {
-      float g = gate[i];
-      for (int p = 1; p < s.parts; ++p) g += gate[p * s.part_stride + i];
-      xt[xs_index(i, ld)] = x[i] * inv * s.norm_w[i] / (1.0f + expf(-g));
+    if (wph > 1) {
+      if (lane == 0) red[warp] = ss;
+      __syncthreads();
+      ss = 0.f;
+      for (int k = 0; k < wph; ++k) ss += red[warp - sub + k];
+      __syncthreads();
     }
+    const float inv = 1.0f / sqrtf(ss / (float)hd + s.eps);
+#pragma unroll 4
+    for (int i = first; i < end; i += step) xt[xs_index(i, ld)] *= inv;
   }
 }
 
@@ -160,7 +174,7 @@ __device__ __forceinline__ void norm_source(const GemvSource& s, int cols, int l
     const float* x = s.x + r * cols;
     float* xt = xs + t * ld;
     if (KIND == GV_GATED_IN) {
-      gate_source(s, x, s.gate + r * s.gate_ld, cols, ld, xt);
+      gate_source(s, x, s.gate + r * s.gate_ld, cols, ld, xt, red);
     } else {
       if (KIND == GV_GROUPS_IN) x = s.x + r * s.x_ld + blockIdx.z * s.x_group;
       const bool step = KIND == GV_ROWS_IN && s.y;
@@ -218,8 +232,9 @@ __global__ void __launch_bounds__(GV_THREADS, sizeof(E) == 2 ? (TT == 1 ? 4 : 3)
   if (KIND == GV_GROUPS_IN) {
     if (cta < a.store_ctas) {
       pdl_launch_dependents();
+      const float2 turn = latent_turn(a.store, cta);
       pdl_wait();
-      if (blockIdx.y == 0 && blockIdx.z == 0) latent_store_row<E>(a.store, cta, red);
+      if (blockIdx.y == 0 && blockIdx.z == 0) latent_store_row<E>(a.store, cta, turn, red);
       return;
     }
     cta -= a.store_ctas;

@@ -38,7 +38,7 @@ struct KvDenseLayer {
 
 // The recurrent state of one layer, f32, per (slot, head, tile of 32 value columns) one record
 //
-//   [ S dim x 32 ][ n dim, rounded up to 4 ][ m, 3 unused ]
+//   [ S dim x 32 ][ n dim, rounded up to 4 ][ m, 3 floats of use inside a step ]
 //
 // with its own copy of n and of the maximum m, so that the tiles of a head need nothing of one
 // another. The state before position 0 is never read.

@@ -65,48 +65,74 @@ __device__ __forceinline__ void latent_out(const LatentRowsArgs& p, int64_t i, i
     static_cast<E*>(p.r.out)[at] = to_elem<E>(v);
 }
 
-// The shares of one head of one row (blockIdx.x, blockIdx.y), four columns per thread.
-constexpr int LM_THREADS = 128;
+// The shares of one head of one row (blockIdx.x, blockIdx.y) in 128 of its columns (blockIdx.z): a
+// thread takes four of them from every eighth share.
+constexpr int LM_THREADS = 256, LM_COLS = 128, LM_GROUPS = LM_THREADS / (LM_COLS / 4);
 template <typename E>
 __global__ void __launch_bounds__(LM_THREADS) latent_merge_kernel(const LatentRowsArgs p) {
-  extern __shared__ float weight[];  // [parts]
+  extern __shared__ float weight[];  // [parts], then the shares' denominators
+  __shared__ __align__(16) float4 sums[LM_GROUPS][LM_COLS / 4];
   pdl_launch_dependents();
-  const int h = blockIdx.x, R = p.a.rank;
+  const int h = blockIdx.x, R = p.a.rank, tid = threadIdx.x;
   const int64_t i = blockIdx.y;
   const uint32_t n = latent_span(p, i, 0).n_parts;
   const float* src = p.partial + ((size_t)i * p.a.heads + h) * p.parts * p.rec;
+  float* dens = weight + p.parts;
+  const int q = tid % (LM_COLS / 4), g = tid / (LM_COLS / 4), c = blockIdx.z * LM_COLS + q * 4;
   pdl_wait();
-  if (threadIdx.x < 32) {
-    const float sink = p.a.sink[h];
-    float top = sink, den = 0.f;
-    for (uint32_t k = threadIdx.x; k < n; k += 32)
-      top = fmaxf(top, src[(size_t)k * p.rec + p.rec - 4]);
+  float4 o[4];
+  // the first shares' sums are on their way while the weights are formed
 #pragma unroll
-    for (int o = 16; o; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xFFFFFFFFu, top, o));
-    for (uint32_t k = threadIdx.x; k < n; k += 32) {
-      const float w = expf(src[(size_t)k * p.rec + p.rec - 4] - top);
-      den += w * src[(size_t)k * p.rec + p.rec - 3];
-      weight[k] = w;
-    }
-#pragma unroll
-    for (int o = 16; o; o >>= 1) den += __shfl_xor_sync(0xFFFFFFFFu, den, o);
-    const float inv = 1.0f / (den + expf(sink - top));
-    for (uint32_t k = threadIdx.x; k < n; k += 32) weight[k] *= inv;
+  for (int k = 0; k < 4; ++k) {
+    const uint32_t at = g + k * LM_GROUPS;
+    o[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (at < n && c < R) o[k] = *reinterpret_cast<const float4*>(src + (size_t)at * p.rec + c);
+  }
+  for (uint32_t k = tid; k < n; k += LM_THREADS) {
+    const float2 m = *reinterpret_cast<const float2*>(src + (size_t)k * p.rec + p.rec - 4);
+    weight[k] = m.x;
+    dens[k] = m.y;
   }
   __syncthreads();
-  for (int c = threadIdx.x * 4; c < R; c += LM_THREADS * 4) {
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
-    for (uint32_t k = 0; k < n; ++k) {
-      const float4 o = *reinterpret_cast<const float4*>(src + (size_t)k * p.rec + c);
-      const float w = weight[k];
-      v.x = fmaf(w, o.x, v.x), v.y = fmaf(w, o.y, v.y);
-      v.z = fmaf(w, o.z, v.z), v.w = fmaf(w, o.w, v.w);
+  if (tid < 32) {
+    const float sink = p.a.sink[h];
+    float top = sink, den = 0.f;
+    for (uint32_t k = tid; k < n; k += 32) top = fmaxf(top, weight[k]);
+#pragma unroll
+    for (int s = 16; s; s >>= 1) top = fmaxf(top, __shfl_xor_sync(0xFFFFFFFFu, top, s));
+    for (uint32_t k = tid; k < n; k += 32) {
+      weight[k] = expf(weight[k] - top);
+      den += weight[k] * dens[k];
     }
-    latent_out<E>(p, i, h, c, v.x);
-    if (c + 1 < R) latent_out<E>(p, i, h, c + 1, v.y);
-    if (c + 2 < R) latent_out<E>(p, i, h, c + 2, v.z);
-    if (c + 3 < R) latent_out<E>(p, i, h, c + 3, v.w);
+#pragma unroll
+    for (int s = 16; s; s >>= 1) den += __shfl_xor_sync(0xFFFFFFFFu, den, s);
+    const float inv = 1.0f / (den + expf(sink - top));
+    for (uint32_t k = tid; k < n; k += 32) weight[k] *= inv;
+  }
+  __syncthreads();
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (uint32_t k0 = g; k0 < n; k0 += 4 * LM_GROUPS) {
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const uint32_t at = k0 + k * LM_GROUPS;
+      const float w = at < n ? weight[at] : 0.f;
+      if (at < n) {  // the pad behind the last column may hold anything
+        v.x = fmaf(w, o[k].x, v.x), v.y = fmaf(w, o[k].y, v.y);
+        v.z = fmaf(w, o[k].z, v.z), v.w = fmaf(w, o[k].w, v.w);
+      }
+      const uint32_t next = at + 4 * LM_GROUPS;
+      if (next < n && c < R)
+        o[k] = *reinterpret_cast<const float4*>(src + (size_t)next * p.rec + c);
+    }
+  }
+  sums[g][q] = v;
+  __syncthreads();
+  const int col = blockIdx.z * LM_COLS + tid;
+  if (tid < LM_COLS && col < R) {
+    float t = 0.f;
+#pragma unroll
+    for (int k = 0; k < LM_GROUPS; ++k) t += reinterpret_cast<const float*>(sums[k])[tid];
+    latent_out<E>(p, i, h, col, t);
   }
 }
 
@@ -513,8 +539,10 @@ static int group_stages(const LatentAttn& a, uint32_t k_dim, size_t* smem) {
   const size_t stage = (size_t)((k_dim + 63) / 64) * LG_PANEL;
   const size_t rest = 1024 + (size_t)16 * (((k_dim + 15u) & ~15u) + 8) * 2 + 4 * 16 * LG_SP * 4 +
                       16 * LG_PS * 2 + (size_t)a.rot * 4;
+  // two CTAs per SM where two stages leave room for it: one's barriers are the other's work
+  const size_t room = 2 * stage + rest <= 110 * 1024 ? 110 * 1024 : 222 * 1024;
   int n = LG_MAX_STAGES;
-  while (n > 0 && n * stage + rest > 222 * 1024) --n;
+  while (n > 0 && n * stage + rest > room) --n;
   *smem = n * stage + rest;
   return n >= 2 ? n : 0;
 }
@@ -600,8 +628,9 @@ int32_t launch_latent_attn_rows(kanso_cuda_ctx* ctx, int32_t compute, const Late
   if (p.parts == 1) return KANSO_OK;
   auto merge =
       compute == KANSO_COMPUTE_BF16 ? latent_merge_kernel<bf16> : latent_merge_kernel<float>;
-  const cudaError_t e = launch_dependent(ctx, merge, dim3(a.heads, (unsigned)r.n),
-                                         dim3(LM_THREADS), (size_t)p.parts * 4, p);
+  const dim3 mgrid(a.heads, (unsigned)r.n, (a.rank + LM_COLS - 1) / LM_COLS);
+  const cudaError_t e =
+      launch_dependent(ctx, merge, mgrid, dim3(LM_THREADS), (size_t)p.parts * 8, p);
   if (e != cudaSuccess) return cuda_fail(ctx, e, "latent merge launch");
   return after_launch(ctx, "latent_merge");
 }

@@ -243,7 +243,20 @@ __global__ void __launch_bounds__(ML_THREADS) mlstm_operands_kernel(const MlstmA
   pdl_wait();
   const int64_t t = blockIdx.x, row = t * a.width();
   const int H = a.heads, D = a.dim, V = a.vdim;
+  const bool four = D % 8 == 0 && V % 8 == 0 && a.width() % 4 == 0 && a.part_stride % 4 == 0;
   auto copy = [&](int64_t from, bf16* to, int n, int ld) {
+    if (four) {  // rows without pads: the heads lie one after the other on both sides
+      for (int i = threadIdx.x * 4; i < H * n; i += ML_THREADS * 4) {
+        float4 v = *reinterpret_cast<const float4*>(a.y + from + i);
+        for (int p = 1; p < a.parts; ++p) {
+          const float4 u = *reinterpret_cast<const float4*>(a.y + p * a.part_stride + from + i);
+          v.x += u.x, v.y += u.y, v.z += u.z, v.w += u.w;
+        }
+        *reinterpret_cast<uint2*>(to + t * H * ld + i) =
+            make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+      }
+      return;
+    }
     for (int i = threadIdx.x * 2; i < H * ld; i += ML_THREADS * 2) {
       const int h = i / ld, d = i - h * ld;
       const float x = d < n ? ml_value(a, from + (int64_t)h * n + d) : 0.f;
@@ -354,7 +367,9 @@ __global__ void __launch_bounds__(McShape<DW, VW, NT, KB>::kThreads, 1)
   for (int i = tid; i < Sh::kDim; i += NTHR)
     ns[i] = !fresh && i < D ? rec0[a.state.n_at() + i] : 0.f;
   // the sequence starts from a maximum of 0, what a segment adds from none
-  float m = pass == kCollect ? -INFINITY : fresh ? 0.f : rec0[a.state.m_at()];
+  float m = pass == kCollect ? -INFINITY
+            : fresh          ? 0.f
+                             : rec0[a.state.m_at() + (pass == kEmit ? 2 : 0)];
   float f_all = 0.f;
 
   constexpr int dc = Sh::kDim / 8;
@@ -654,43 +669,57 @@ __global__ void __launch_bounds__(McShape<DW, VW, NT, KB>::kThreads, 1)
 }
 
 // The state in front of every segment of a portion, in place of what the segment before it adds;
-// blockIdx = (tile, head, portion).
+// blockIdx = (tile and part of its record, head, portion). The maxima in front go to places of
+// their own (m_at() + 2): the segments' own are read by other CTAs.
+constexpr int MS_PARTS = 4, MS_AHEAD = 4;
 __global__ void __launch_bounds__(ML_THREADS) mlstm_scan_kernel(const MlstmArgs a,
                                                                const MlSegments seg) {
   pdl_launch_dependents();
   pdl_wait();
   const MlPortion p = ml_portion(a, blockIdx.z);
   const uint32_t n = (p.rows + seg.rows - 1) / seg.rows, at_m = a.state.m_at();
+  const uint32_t tile = blockIdx.x / MS_PARTS, part = blockIdx.x % MS_PARTS;
   const bool fresh = p.pos0 == 0;
-  const float* start = a.state.at(p.slot, blockIdx.y, blockIdx.x);
+  const float* start = a.state.at(p.slot, blockIdx.y, tile);
   const float m0 = fresh ? 0.f : start[at_m];
-  auto rec = [&](uint32_t s) {
-    return seg.state.at(blockIdx.z * seg.n + s, blockIdx.y, blockIdx.x);
-  };
-  for (uint32_t i = threadIdx.x * 4; i < at_m; i += ML_THREADS * 4) {
+  const size_t step = seg.state.slot_floats();
+  float* base = seg.state.at(blockIdx.z * seg.n, blockIdx.y, tile);
+  for (uint32_t i = (part * ML_THREADS + threadIdx.x) * 4; i < at_m;
+       i += MS_PARTS * ML_THREADS * 4) {
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (!fresh) v = *reinterpret_cast<const float4*>(start + i);
-    *reinterpret_cast<float4*>(rec(0) + i) = v;
+    *reinterpret_cast<float4*>(base + i) = v;
     float m = m0;
-    for (uint32_t s = 1; s < n; ++s) {
-      float* r = rec(s);
-      const float add = r[at_m], f = r[at_m + 1], top = fmaxf(f + m, add);
-      const float keep = expf(f + m - top), take = expf(add - top);
-      const float4 u = *reinterpret_cast<const float4*>(r + i);
-      v.x = fmaf(keep, v.x, take * u.x), v.y = fmaf(keep, v.y, take * u.y);
-      v.z = fmaf(keep, v.z, take * u.z), v.w = fmaf(keep, v.w, take * u.w);
-      *reinterpret_cast<float4*>(r + i) = v;
-      m = top;
+    for (uint32_t s0 = 1; s0 < n; s0 += MS_AHEAD) {
+      float4 u[MS_AHEAD];
+      float add[MS_AHEAD], f[MS_AHEAD];
+#pragma unroll
+      for (int k = 0; k < MS_AHEAD; ++k)
+        if (s0 + k < n) {
+          const float* r = base + (s0 + k) * step;
+          u[k] = *reinterpret_cast<const float4*>(r + i);
+          add[k] = r[at_m];
+          f[k] = r[at_m + 1];
+        }
+#pragma unroll
+      for (int k = 0; k < MS_AHEAD; ++k)
+        if (s0 + k < n) {
+          const float top = fmaxf(f[k] + m, add[k]);
+          const float keep = expf(f[k] + m - top), take = expf(add[k] - top);
+          v.x = fmaf(keep, v.x, take * u[k].x), v.y = fmaf(keep, v.y, take * u[k].y);
+          v.z = fmaf(keep, v.z, take * u[k].z), v.w = fmaf(keep, v.w, take * u[k].w);
+          *reinterpret_cast<float4*>(base + (s0 + k) * step + i) = v;
+          m = top;
+        }
     }
   }
-  __syncthreads();  // the segments' own maxima have been read
-  if (threadIdx.x == 0) {
+  if (part == 0 && threadIdx.x == 0) {
     float m = m0;
-    rec(0)[at_m] = m;
+    base[at_m + 2] = m;
     for (uint32_t s = 1; s < n; ++s) {
-      float* r = rec(s);
+      float* r = base + s * step;
       m = fmaxf(r[at_m + 1] + m, r[at_m]);
-      r[at_m] = m;
+      r[at_m + 2] = m;
     }
   }
 }
@@ -767,7 +796,7 @@ static int32_t chunk_launch(kanso_cuda_ctx* ctx, const MlstmArgs& a, const MlOpe
   if (!seg.state.base) return KANSO_ERR_DEVICE;
   int32_t st = pass(seg, kCollect);
   if (!st)
-    st = ml_launch(ctx, mlstm_scan_kernel, dim3(a.state.tiles(), a.heads, n), 0, "mlstm_scan",
+    st = ml_launch(ctx, mlstm_scan_kernel, dim3(a.state.tiles() * MS_PARTS, a.heads, n), 0, "mlstm_scan",
                    ML_THREADS, a, seg);
   return st ? st : pass(seg, kEmit);
 }

@@ -3,8 +3,9 @@
 // part (rotated columns) of which the keys' is shared by all heads; the softmax's denominator may
 // hold one more term per head that has no key and no value (a sink).
 //
-//   warp 8     copies by tensor map: the query tile once, then a two-stage ring of key and value
-//              tiles in panels of 64 columns (128-byte swizzle)
+//   warps 8, 10  copies by tensor map, panels of 64 columns (128-byte swizzle): the query tile once
+//              and a ring of key tiles; a ring of value tiles. Two warps, since a value tile's place
+//              is free much later than a key tile's, which would wait behind it.
 //   warp 9     issues S = Q K^T (M = 128, N = 64) into one of two score buffers and, for the tile
 //              before, O += P V (V N-major) into one of two output accumulators
 //   warps 0-7  two groups of four, each with a score buffer, a weight buffer and an output
@@ -22,8 +23,8 @@
 
 namespace kanso {
 
-constexpr int SX_Q = 128, SX_K = 64, SX_STAGES = 2;
-constexpr int SX_WORKERS = 256, SX_THREADS = 320;
+constexpr int SX_Q = 128, SX_K = 64, SX_MAX_STAGES = 4;
+constexpr int SX_WORKERS = 256, SX_THREADS = 352;
 constexpr int SX_P_BYTES = SX_Q * SX_K * 2;
 constexpr float SX_SLACK = 8.f;
 
@@ -36,6 +37,7 @@ struct SoftmaxArgs {
   int v_dim, nv, o_step;   // nv: v_dim rounded up to 16; o_step: to 32, between the accumulators
   int k_panels, r_panels, v_panels;  // 64-column panels of K, of its second part and of V
   int k_steps, r_steps;    // 16-column steps of the scores
+  int k_stages, v_stages;
   uint32_t tmem_cols;
   int* status;
 };
@@ -47,8 +49,8 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
                            const __grid_constant__ CUtensorMap krmap,
                            const __grid_constant__ CUtensorMap vmap, const SoftmaxArgs p) {
   extern __shared__ uint8_t raw[];
-  __shared__ uint64_t q_full, k_full[SX_STAGES], k_empty[SX_STAGES], v_full[SX_STAGES],
-      v_empty[SX_STAGES], s_full[2], s_free[2], p_full[2], p_free[2], o_full;
+  __shared__ uint64_t q_full, k_full[SX_MAX_STAGES], k_empty[SX_MAX_STAGES],
+      v_full[SX_MAX_STAGES], v_empty[SX_MAX_STAGES], s_full[2], s_free[2], p_full[2], p_free[2], o_full;
   __shared__ uint32_t tmem_slot;
   __shared__ volatile int abort_flag;
   __shared__ float2 ml[2][SX_Q];  // per group and row: reference maximum, denominator
@@ -60,14 +62,14 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
   const uint32_t q_panel = SX_Q * 128u;
   uint8_t* Qs = raw + ((1024u - (smem_u32(raw) & 1023u)) & 1023u);
   uint8_t* Ks = Qs + (size_t)panels * q_panel;
-  uint8_t* Vs = Ks + (size_t)SX_STAGES * k_bytes;
-  uint8_t* Ps = Vs + (size_t)SX_STAGES * v_bytes;
+  uint8_t* Vs = Ks + (size_t)p.k_stages * k_bytes;
+  uint8_t* Ps = Vs + (size_t)p.v_stages * v_bytes;
 
   pdl_launch_dependents();
   if (tid == 0) {
     mbar_init(&q_full, 1);
     mbar_init(&o_full, 1);
-    for (int i = 0; i < SX_STAGES; ++i) {
+    for (int i = 0; i < SX_MAX_STAGES; ++i) {
       mbar_init(&k_full[i], 1);
       mbar_init(&k_empty[i], 1);
       mbar_init(&v_full[i], 1);
@@ -95,41 +97,38 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
   tc_fence_after();
   const uint32_t tmem = tmem_slot, o_tmem = tmem + 2 * SX_K;
 
-  if (warp == 8) {
+  if (warp == 8 || warp == 10) {
     // ---- copies ----
     if (lane == 0) {
-      mbar_arrive_expect_tx(&q_full, (uint32_t)panels * q_panel);
-      for (int c = 0; c < panels; ++c) {
-        const bool second = c >= p.k_panels;
-        tma_load_3d(Qs + (size_t)c * q_panel, second ? &qrmap : &qmap,
-                    (second ? c - p.k_panels : c) * 64, h, (int)tile.row0, &q_full);
+      const bool keys = warp == 8;
+      const int stages = keys ? p.k_stages : p.v_stages;
+      const uint32_t bytes = keys ? k_bytes : v_bytes;
+      uint64_t *full = keys ? k_full : v_full, *empty = keys ? k_empty : v_empty;
+      if (keys) {
+        mbar_arrive_expect_tx(&q_full, (uint32_t)panels * q_panel);
+        for (int c = 0; c < panels; ++c) {
+          const bool second = c >= p.k_panels;
+          tma_load_3d(Qs + (size_t)c * q_panel, second ? &qrmap : &qmap,
+                      (second ? c - p.k_panels : c) * 64, h, (int)tile.row0, &q_full);
+        }
       }
-      int k_issued = 0, v_issued = 0;
+      int issued = 0;
       for (int i = 0; i < n_tiles; ++i) {
-        const int s = i % SX_STAGES;
-        const uint32_t par = ((uint32_t)(i / SX_STAGES) & 1u) ^ 1u;
-        if (!mbar_wait_abort(&k_empty[s], par, &abort_flag)) break;
-        mbar_arrive_expect_tx(&k_full[s], k_bytes);
-        uint8_t* kd = Ks + (size_t)s * k_bytes;
-        for (int c = 0; c < p.k_panels; ++c)
-          tma_load_3d(kd + (size_t)c * SX_K * 128, &kmap, c * 64, h, key0 + i * SX_K, &k_full[s]);
-        for (int c = 0; c < p.r_panels; ++c)
-          tma_load_2d(kd + (size_t)(p.k_panels + c) * SX_K * 128, &krmap, c * 64, key0 + i * SX_K,
-                      &k_full[s]);
-        k_issued = i + 1;
-        if (!mbar_wait_abort(&v_empty[s], par, &abort_flag)) break;
-        mbar_arrive_expect_tx(&v_full[s], v_bytes);
-        for (int c = 0; c < p.v_panels; ++c)
-          tma_load_3d(Vs + (size_t)s * v_bytes + (size_t)c * SX_K * 128, &vmap, c * 64, h,
-                      key0 + i * SX_K, &v_full[s]);
-        v_issued = i + 1;
+        const int s = i % stages;
+        if (!mbar_wait_abort(&empty[s], ((uint32_t)(i / stages) & 1u) ^ 1u, &abort_flag)) break;
+        mbar_arrive_expect_tx(&full[s], bytes);
+        uint8_t* dst = (keys ? Ks : Vs) + (size_t)s * bytes;
+        const int row = key0 + i * SX_K;
+        for (int c = 0; c < (keys ? p.k_panels : p.v_panels); ++c)
+          tma_load_3d(dst + (size_t)c * SX_K * 128, keys ? &kmap : &vmap, c * 64, h, row, &full[s]);
+        for (int c = 0; keys && c < p.r_panels; ++c)
+          tma_load_2d(dst + (size_t)(p.k_panels + c) * SX_K * 128, &krmap, c * 64, row, &full[s]);
+        issued = i + 1;
       }
       // leave only when every copy has landed (bounded)
-      mbar_wait_bounded(&q_full, 0);
-      for (int i = max(0, k_issued - SX_STAGES); i < k_issued; ++i)
-        mbar_wait_bounded(&k_full[i % SX_STAGES], (uint32_t)(i / SX_STAGES) & 1u);
-      for (int i = max(0, v_issued - SX_STAGES); i < v_issued; ++i)
-        mbar_wait_bounded(&v_full[i % SX_STAGES], (uint32_t)(i / SX_STAGES) & 1u);
+      if (keys) mbar_wait_bounded(&q_full, 0);
+      for (int i = max(0, issued - stages); i < issued; ++i)
+        mbar_wait_bounded(&full[i % stages], (uint32_t)(i / stages) & 1u);
     }
     __syncwarp();
   } else if (warp == 9) {
@@ -139,8 +138,8 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
       const uint32_t id_o = tc_idesc_bf16(SX_Q, p.nv) | (1u << 16);  // B is N-major
       bool ok = mbar_wait_abort(&q_full, 0, &abort_flag);
       auto scores = [&](int i) {
-        const int s = i % SX_STAGES;
-        if (ok) ok = mbar_wait_abort(&k_full[s], (uint32_t)(i / SX_STAGES) & 1u, &abort_flag);
+        const int s = i % p.k_stages;
+        if (ok) ok = mbar_wait_abort(&k_full[s], (uint32_t)(i / p.k_stages) & 1u, &abort_flag);
         if (!ok) return;
         tc_fence_after();
         const uint32_t q0 = smem_u32(Qs), k0 = smem_u32(Ks) + (uint32_t)s * k_bytes;
@@ -158,7 +157,7 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
       scores(0);
       if (n_tiles > 1) scores(1);
       for (int i = 0; i < n_tiles && ok; ++i) {
-        const int b = i & 1, s = i % SX_STAGES;
+        const int b = i & 1, s = i % p.v_stages;
         const uint32_t par = (uint32_t)(i >> 1) & 1u;
         if (i + 2 < n_tiles) {
           ok = mbar_wait_abort(&s_free[b], par, &abort_flag);
@@ -166,7 +165,7 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
           tc_fence_after();
           scores(i + 2);
         }
-        if (ok) ok = mbar_wait_abort(&v_full[s], (uint32_t)(i / SX_STAGES) & 1u, &abort_flag);
+        if (ok) ok = mbar_wait_abort(&v_full[s], (uint32_t)(i / p.v_stages) & 1u, &abort_flag);
         if (ok) ok = mbar_wait_abort(&p_full[b], par, &abort_flag);
         if (!ok) break;
         tc_fence_after();
@@ -304,14 +303,24 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
   if (warp == 9) tmem_dealloc(tmem, p.tmem_cols);
 }
 
-static size_t softmax_smem(const SoftmaxPrefill& p) {
+// Stages of the two rings and the shared memory they come to; false: two of each do not fit.
+static bool softmax_stages(const SoftmaxPrefill& p, int* k_stages, int* v_stages, size_t* smem) {
   const size_t kp = (p.dim + 63) / 64 + (p.rot + 63) / 64, vp = (p.vdim + 63) / 64;
-  return 1024 + kp * SX_Q * 128 + (size_t)SX_STAGES * SX_K * 128 * (kp + vp) + 2 * SX_P_BYTES;
+  const size_t fixed = 1024 + kp * SX_Q * 128 + 2 * SX_P_BYTES, one = (size_t)SX_K * 128;
+  int k = SX_MAX_STAGES, v = SX_MAX_STAGES;
+  while (k > 2 && fixed + one * (k * kp + v * vp) > 222 * 1024) k >= v ? --k : --v;
+  if (k == 2) v = std::min(v, 2);
+  *k_stages = k;
+  *v_stages = v;
+  *smem = fixed + one * (k * kp + v * vp);
+  return *smem <= 222 * 1024;
 }
 
 bool softmax_prefill_fits(const SoftmaxPrefill& p) {
+  int k = 0, v = 0;
+  size_t smem = 0;
   return p.dim && p.vdim && p.vdim <= 192 && p.heads <= 65535 && p.scale > 0.f &&
-         p.keys < (1 << 30) && softmax_smem(p) <= 222 * 1024 && tm_encoder();
+         p.keys < (1 << 30) && softmax_stages(p, &k, &v, &smem) && tm_encoder();
 }
 
 int32_t launch_softmax_prefill(kanso_cuda_ctx* ctx, const SoftmaxPrefill& p, bool* handled) {
@@ -334,6 +343,8 @@ int32_t launch_softmax_prefill(kanso_cuda_ctx* ctx, const SoftmaxPrefill& p, boo
   a.r_steps = (int)((p.rot + 15u) / 16u);
   a.tmem_cols = 2 * SX_K + 2 * a.o_step <= 256 ? 256 : 512;
   a.status = ctx->dev_status;
+  size_t smem = 0;
+  softmax_stages(p, &a.k_stages, &a.v_stages, &smem);
   const uint64_t dl = round_up8(p.dim), vl = round_up8(p.vdim), rl = round_up8(p.rot), H = p.heads;
   CUtensorMap qm, qrm, km, krm, vm;
   bool ok = tm_map3(encode, p.q, dl, H, (uint64_t)p.q_rows, dl, H * dl, 1, SX_Q, &qm) &&
@@ -349,7 +360,7 @@ int32_t launch_softmax_prefill(kanso_cuda_ctx* ctx, const SoftmaxPrefill& p, boo
   if (st) return st;
   *handled = true;
   const cudaError_t e = launch_dependent(ctx, softmax_prefill_kernel, dim3(p.n_tiles, p.heads),
-                                         dim3(SX_THREADS), softmax_smem(p), qm, qrm, km, krm, vm, a);
+                                         dim3(SX_THREADS), smem, qm, qrm, km, krm, vm, a);
   if (e != cudaSuccess) return cuda_fail(ctx, e, "softmax prefill launch");
   return after_launch(ctx, "softmax_prefill");
 }
