@@ -55,7 +55,7 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
   __shared__ volatile int abort_flag;
   __shared__ float2 ml[2][SX_Q];  // per group and row: reference maximum, denominator
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int h = blockIdx.y;
+  const int h = blockIdx.x;
   const int panels = p.k_panels + p.r_panels;
   const uint32_t k_bytes = (uint32_t)panels * SX_K * 128u;
   const uint32_t v_bytes = (uint32_t)p.v_panels * SX_K * 128u;
@@ -77,15 +77,15 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
     }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&s_full[i], 1);
-      mbar_init(&s_free[i], SX_WORKERS / 2);
-      mbar_init(&p_full[i], SX_WORKERS / 2);
+      mbar_init(&s_free[i], SX_WORKERS / 64);
+      mbar_init(&p_full[i], SX_WORKERS / 64);
       mbar_init(&p_free[i], 1);
     }
     mbar_fence_init();
     abort_flag = 0;
   }
-  // the longest rows first: their CTAs start while others are still to come
-  const AttnTile tile = p.tiles[gridDim.x - 1 - blockIdx.x];
+  // the longest rows of all heads first: what is left at the end is short
+  const AttnTile tile = p.tiles[gridDim.y - 1 - blockIdx.y];
   const int key0 = (int)tile.seq;
   const int q_end = (int)(tile.pos0 + tile.rows);  // exclusive
   const int n_tiles = (q_end + SX_K - 1) / SX_K;
@@ -136,21 +136,20 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
     if (lane == 0) {
       const uint32_t id_s = tc_idesc_bf16(SX_Q, SX_K);
       const uint32_t id_o = tc_idesc_bf16(SX_Q, p.nv) | (1u << 16);  // B is N-major
+      const uint32_t queries = smem_u32(Qs), keys = smem_u32(Ks);
+      const uint64_t weights = tc_smem_desc_sw128(smem_u32(Ps));
+      const uint64_t values = tc_smem_desc_nmajor(smem_u32(Vs), SX_K * 128u);
       bool ok = mbar_wait_abort(&q_full, 0, &abort_flag);
       auto scores = [&](int i) {
         const int s = i % p.k_stages;
         if (ok) ok = mbar_wait_abort(&k_full[s], (uint32_t)(i / p.k_stages) & 1u, &abort_flag);
         if (!ok) return;
         tc_fence_after();
-        const uint32_t q0 = smem_u32(Qs), k0 = smem_u32(Ks) + (uint32_t)s * k_bytes;
-        for (int k = 0; k < p.k_steps + p.r_steps; ++k) {
-          const bool second = k >= p.k_steps;
-          const uint32_t step = (uint32_t)(second ? k - p.k_steps : k);
-          const uint32_t panel = (second ? (uint32_t)p.k_panels : 0u) + (step >> 2);
-          const uint32_t in = (step & 3u) * 2u;
-          tc_mma_f16(tmem + (uint32_t)(i & 1) * SX_K, tc_smem_desc_sw128(q0 + panel * q_panel) + in,
-                     tc_smem_desc_sw128(k0 + panel * (SX_K * 128u)) + in, id_s, k > 0);
-        }
+        const uint32_t k0 = keys + (uint32_t)s * k_bytes, acc = tmem + (uint32_t)(i & 1) * SX_K;
+        tc_mma_panels(acc, queries, k0, q_panel, SX_K * 128u, p.k_steps, id_s, 0);
+        tc_mma_panels(acc, queries + (uint32_t)p.k_panels * q_panel,
+                      k0 + (uint32_t)p.k_panels * (SX_K * 128u), q_panel, SX_K * 128u, p.r_steps,
+                      id_s, 1);
         tc_commit(&k_empty[s]);
         tc_commit(&s_full[i & 1]);
       };
@@ -169,9 +168,8 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
         if (ok) ok = mbar_wait_abort(&p_full[b], par, &abort_flag);
         if (!ok) break;
         tc_fence_after();
-        const uint64_t ad = tc_smem_desc_sw128(smem_u32(Ps) + (uint32_t)b * SX_P_BYTES);
-        const uint64_t bd =
-            tc_smem_desc_nmajor(smem_u32(Vs) + (uint32_t)s * v_bytes, SX_K * 128u);
+        const uint64_t ad = weights + (uint32_t)b * (SX_P_BYTES >> 4);
+        const uint64_t bd = values + (uint32_t)s * (v_bytes >> 4);
 #pragma unroll
         for (int k = 0; k < SX_K / 16; ++k)
           tc_mma_f16(o_tmem + (uint32_t)(b * p.o_step), ad + 2 * k, bd + 128 * k, id_o,
@@ -203,7 +201,8 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
       tmem_ld32(s_lane, r[0]);
       tmem_ld32(s_lane + 32, r[1]);
       tc_fence_before();
-      mbar_arrive(&s_free[wg]);
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&s_free[wg]);
       if (i * SX_K + SX_K - 1 > (int)tile.pos0) {  // some row does not see all of the tile
         const int seen = pos - i * SX_K;
 #pragma unroll
@@ -250,7 +249,8 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
       }
       tc_fence_before();
       fence_proxy_async_smem();
-      mbar_arrive(&p_full[wg]);
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_full[wg]);
     }
     ml[wg][row] = make_float2(ref, l);
   }
@@ -319,7 +319,7 @@ static bool softmax_stages(const SoftmaxPrefill& p, int* k_stages, int* v_stages
 bool softmax_prefill_fits(const SoftmaxPrefill& p) {
   int k = 0, v = 0;
   size_t smem = 0;
-  return p.dim && p.vdim && p.vdim <= 192 && p.heads <= 65535 && p.scale > 0.f &&
+  return p.dim && p.vdim && p.vdim <= 192 && p.n_tiles <= 65535 && p.scale > 0.f &&
          p.keys < (1 << 30) && softmax_stages(p, &k, &v, &smem) && tm_encoder();
 }
 
@@ -359,7 +359,7 @@ int32_t launch_softmax_prefill(kanso_cuda_ctx* ctx, const SoftmaxPrefill& p, boo
   int32_t st = allow_max_smem(ctx, (const void*)softmax_prefill_kernel);
   if (st) return st;
   *handled = true;
-  const cudaError_t e = launch_dependent(ctx, softmax_prefill_kernel, dim3(p.n_tiles, p.heads),
+  const cudaError_t e = launch_dependent(ctx, softmax_prefill_kernel, dim3(p.heads, p.n_tiles),
                                          dim3(SX_THREADS), smem, qm, qrm, km, krm, vm, a);
   if (e != cudaSuccess) return cuda_fail(ctx, e, "softmax prefill launch");
   return after_launch(ctx, "softmax_prefill");

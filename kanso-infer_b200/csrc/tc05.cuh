@@ -163,4 +163,27 @@ __device__ __forceinline__ uint64_t tc_smem_desc_nmajor(uint32_t addr, uint32_t 
   return d;
 }
 
+// One product over operands that lie in panels of 64 columns in the 128-byte swizzle: `steps` of
+// 16 columns from the tiles at shared-memory addresses a and b on, panels a_panel and b_panel bytes
+// apart. The issuing thread is alone with this: what it computes per instruction is one addition.
+__device__ __forceinline__ void tc_mma_panels(uint32_t d_tmem, uint32_t a, uint32_t b,
+                                              uint32_t a_panel, uint32_t b_panel, int steps,
+                                              uint32_t idesc, uint32_t accumulate) {
+  const uint64_t desc = tc_smem_desc_sw128(0);
+  const uint32_t lo = (uint32_t)desc, hi = (uint32_t)(desc >> 32);
+  uint32_t al = lo + (a >> 4), bl = lo + (b >> 4);
+  for (; steps > 0; steps -= 4) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      if (j < steps) {
+        tc_mma_f16(d_tmem, tc_desc_join(al + 2 * j, hi), tc_desc_join(bl + 2 * j, hi), idesc,
+                   accumulate);
+        accumulate = 1;
+      }
+    }
+    al += a_panel >> 4;
+    bl += b_panel >> 4;
+  }
+}
+
 }  // namespace kanso

@@ -47,7 +47,13 @@ ATTENTION = config(77, 72, [latent(6, 32, 16, 24, 40, 48, None), latent(2, 8, 8,
 MEMORY = config(101, 64, [memory(4, 16, 32, dense(50)), memory(2, 33, 31, moe(9, 4, 24))])
 WIDE = config(301, 320, [latent(20, 72, 64, 136, 264, 150, moe(16, 4, 128)),
                          memory(3, 160, 200, dense(400)), memory(2, 270, 96, None)])
-MODELS = {"attention": ATTENTION, "memory": MEMORY, "mixed": MIXED, "one": ONE, "uneven": UNEVEN,
+# nothing here is a multiple of four
+ODD = config(67, 45, [memory(3, 7, 9, dense(21)), latent(3, 9, 6, 11, 13, 11, moe(5, 2, 19)),
+                      memory(1, 35, 33, moe(3, 1, 13)), latent(1, 7, 2, 5, 9, 7, dense(17))])
+# value columns beyond the prompt attention's, key columns beyond the chunks': other kernels step in
+LARGE = config(90, 64, [latent(3, 24, 8, 200, 40, 32, dense(64)), memory(1, 530, 24, None),
+                        latent(2, 360, 16, 16, 24, 16, None)])
+MODELS = {"attention": ATTENTION, "large": LARGE, "odd": ODD, "memory": MEMORY, "mixed": MIXED, "one": ONE, "uneven": UNEVEN,
           "wide": WIDE}
 
 
