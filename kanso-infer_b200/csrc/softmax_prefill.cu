@@ -6,8 +6,9 @@
 //   warps 8, 10  copies by tensor map, panels of 64 columns (128-byte swizzle): the query tile once
 //              and a ring of key tiles; a ring of value tiles. Two warps, since a value tile's place
 //              is free much later than a key tile's, which would wait behind it.
-//   warp 9     issues S = Q K^T (M = 128, N = 64) into one of two score buffers and, for the tile
-//              before, O += P V (V N-major) into one of two output accumulators
+//   warp 9     issues S = Q K^T (M = 128, N = 64) into one of two score buffers
+//   warp 11    issues O += P V (V N-major) into one of two output accumulators. A thread of its own:
+//              in turns with the scores' it would spend a tile's time on waits and issues alone.
 //   warps 0-7  two groups of four, each with a score buffer, a weight buffer and an output
 //              accumulator of its own: group g takes every second tile. A thread owns a query row.
 //
@@ -24,7 +25,7 @@
 namespace kanso {
 
 constexpr int SX_Q = 128, SX_K = 64, SX_MAX_STAGES = 4;
-constexpr int SX_WORKERS = 256, SX_THREADS = 352;
+constexpr int SX_WORKERS = 256, SX_THREADS = 384;
 constexpr int SX_P_BYTES = SX_Q * SX_K * 2;
 constexpr float SX_SLACK = 8.f;
 
@@ -132,50 +133,50 @@ __global__ void __launch_bounds__(SX_THREADS, 1)
     }
     __syncwarp();
   } else if (warp == 9) {
-    // ---- products ----
+    // ---- scores ----
     if (lane == 0) {
-      const uint32_t id_s = tc_idesc_bf16(SX_Q, SX_K);
-      const uint32_t id_o = tc_idesc_bf16(SX_Q, p.nv) | (1u << 16);  // B is N-major
+      const uint32_t idesc = tc_idesc_bf16(SX_Q, SX_K);
       const uint32_t queries = smem_u32(Qs), keys = smem_u32(Ks);
-      const uint64_t weights = tc_smem_desc_sw128(smem_u32(Ps));
-      const uint64_t values = tc_smem_desc_nmajor(smem_u32(Vs), SX_K * 128u);
       bool ok = mbar_wait_abort(&q_full, 0, &abort_flag);
-      auto scores = [&](int i) {
-        const int s = i % p.k_stages;
+      for (int i = 0; i < n_tiles && ok; ++i) {
+        const int b = i & 1, s = i % p.k_stages;
+        // the group has read the scores of the tile before
+        if (i >= 2) ok = mbar_wait_abort(&s_free[b], ((uint32_t)(i >> 1) & 1u) ^ 1u, &abort_flag);
         if (ok) ok = mbar_wait_abort(&k_full[s], (uint32_t)(i / p.k_stages) & 1u, &abort_flag);
-        if (!ok) return;
+        if (!ok) break;
         tc_fence_after();
-        const uint32_t k0 = keys + (uint32_t)s * k_bytes, acc = tmem + (uint32_t)(i & 1) * SX_K;
-        tc_mma_panels(acc, queries, k0, q_panel, SX_K * 128u, p.k_steps, id_s, 0);
+        const uint32_t k0 = keys + (uint32_t)s * k_bytes, acc = tmem + (uint32_t)b * SX_K;
+        tc_mma_panels(acc, queries, k0, q_panel, SX_K * 128u, p.k_steps, idesc, 0);
         tc_mma_panels(acc, queries + (uint32_t)p.k_panels * q_panel,
                       k0 + (uint32_t)p.k_panels * (SX_K * 128u), q_panel, SX_K * 128u, p.r_steps,
-                      id_s, 1);
+                      idesc, 1);
+        tc_commit(&s_full[b]);
         tc_commit(&k_empty[s]);
-        tc_commit(&s_full[i & 1]);
-      };
-      scores(0);
-      if (n_tiles > 1) scores(1);
+      }
+      if (!ok) abort_flag = 1;
+    }
+    __syncwarp();
+  } else if (warp == 11) {
+    // ---- weights x values ----
+    if (lane == 0) {
+      const uint32_t idesc = tc_idesc_bf16(SX_Q, p.nv) | (1u << 16);  // B is N-major
+      const uint64_t weights = tc_smem_desc_sw128(smem_u32(Ps));
+      const uint64_t values = tc_smem_desc_nmajor(smem_u32(Vs), SX_K * 128u);
+      bool ok = true;
       for (int i = 0; i < n_tiles && ok; ++i) {
         const int b = i & 1, s = i % p.v_stages;
-        const uint32_t par = (uint32_t)(i >> 1) & 1u;
-        if (i + 2 < n_tiles) {
-          ok = mbar_wait_abort(&s_free[b], par, &abort_flag);
-          if (!ok) break;
-          tc_fence_after();
-          scores(i + 2);
-        }
-        if (ok) ok = mbar_wait_abort(&v_full[s], (uint32_t)(i / p.v_stages) & 1u, &abort_flag);
-        if (ok) ok = mbar_wait_abort(&p_full[b], par, &abort_flag);
+        ok = mbar_wait_abort(&v_full[s], (uint32_t)(i / p.v_stages) & 1u, &abort_flag);
+        if (ok) ok = mbar_wait_abort(&p_full[b], (uint32_t)(i >> 1) & 1u, &abort_flag);
         if (!ok) break;
         tc_fence_after();
         const uint64_t ad = weights + (uint32_t)b * (SX_P_BYTES >> 4);
         const uint64_t bd = values + (uint32_t)s * (v_bytes >> 4);
+        const uint32_t acc = o_tmem + (uint32_t)(b * p.o_step);
+        tc_mma_f16(acc, ad, bd, idesc, i > 1);
 #pragma unroll
-        for (int k = 0; k < SX_K / 16; ++k)
-          tc_mma_f16(o_tmem + (uint32_t)(b * p.o_step), ad + 2 * k, bd + 128 * k, id_o,
-                     (i > 1 || k > 0) ? 1u : 0u);
-        tc_commit(&v_empty[s]);
+        for (int k = 1; k < SX_K / 16; ++k) tc_mma_f16(acc, ad + 2 * k, bd + 128 * k, idesc, 1);
         tc_commit(&p_free[b]);
+        tc_commit(&v_empty[s]);
       }
       if (ok)
         tc_commit(&o_full);

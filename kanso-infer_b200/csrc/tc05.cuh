@@ -172,17 +172,19 @@ __device__ __forceinline__ void tc_mma_panels(uint32_t d_tmem, uint32_t a, uint3
   const uint64_t desc = tc_smem_desc_sw128(0);
   const uint32_t lo = (uint32_t)desc, hi = (uint32_t)(desc >> 32);
   uint32_t al = lo + (a >> 4), bl = lo + (b >> 4);
-  for (; steps > 0; steps -= 4) {
+  for (; steps >= 4; steps -= 4) {
+    tc_mma_f16(d_tmem, tc_desc_join(al, hi), tc_desc_join(bl, hi), idesc, accumulate);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      if (j < steps) {
-        tc_mma_f16(d_tmem, tc_desc_join(al + 2 * j, hi), tc_desc_join(bl + 2 * j, hi), idesc,
-                   accumulate);
-        accumulate = 1;
-      }
-    }
+    for (int j = 1; j < 4; ++j)
+      tc_mma_f16(d_tmem, tc_desc_join(al + 2 * j, hi), tc_desc_join(bl + 2 * j, hi), idesc, 1);
+    accumulate = 1;
     al += a_panel >> 4;
     bl += b_panel >> 4;
+  }
+  for (int j = 0; j < steps; ++j) {
+    tc_mma_f16(d_tmem, tc_desc_join(al + 2 * j, hi), tc_desc_join(bl + 2 * j, hi), idesc,
+               accumulate);
+    accumulate = 1;
   }
 }
 
