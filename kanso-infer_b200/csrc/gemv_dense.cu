@@ -14,6 +14,7 @@
 // experts' one after the other. A matrix of several groups (one per head) takes an input of its own
 // for each.
 #include <cmath>
+#include <type_traits>
 
 #include "dense.cuh"
 
@@ -115,9 +116,10 @@ __device__ __forceinline__ void finish_rows(float (&acc)[V], int ks, float* red,
   __syncthreads();
 }
 
-// What a launch of the plain product's kernel is made for: rows with the residual step, inputs that
-// lie in groups (and the store beside them), or gated heads.
-enum GemvKind { GV_ROWS_IN, GV_GROUPS_IN, GV_GATED_IN };
+// What a launch of the plain product's kernel is made for: rows with a residual step that adds and
+// results as they are; rows with any residual step and results through GemvOut; inputs that lie in
+// groups (and the store beside them); gated heads.
+enum GemvKind { GV_PLAIN, GV_ROWS_IN, GV_GROUPS_IN, GV_GATED_IN };
 
 struct GemvArgs {
   const void* w;
@@ -126,9 +128,13 @@ struct GemvArgs {
   float* out;
   int64_t out_ld;
   GemvOut o;
+};
+struct GemvStoreArgs : GemvArgs {
   int store_ctas;  // CTAs in front of the product's that store the step's cache rows
   LatentStore store;
 };
+template <int KIND>
+using GemvArgsOf = std::conditional_t<KIND == GV_GROUPS_IN, GemvStoreArgs, GemvArgs>;
 
 // Each head over its own root mean square, weight and gate (GemvSource::gate): a warp per head, or
 // several where the heads are few. Every thread of the CTA must come here.
@@ -177,8 +183,8 @@ __device__ __forceinline__ void norm_source(const GemvSource& s, int cols, int l
       gate_source(s, x, s.gate + r * s.gate_ld, cols, ld, xt, red);
     } else {
       if (KIND == GV_GROUPS_IN) x = s.x + r * s.x_ld + blockIdx.z * s.x_group;
-      const bool step = KIND == GV_ROWS_IN && s.y;
-      const bool after = step && s.form == Residual::kAddNorm;
+      const bool step = KIND != GV_GROUPS_IN && s.y;
+      const bool after = KIND == GV_ROWS_IN && step && s.form == Residual::kAddNorm;
       float inv = 0.f;
       if (step) {
         const float* y = s.y + r * cols;
@@ -219,7 +225,7 @@ __device__ __forceinline__ void norm_source(const GemvSource& s, int cols, int l
 
 template <typename E, int TT, int KIND>
 __global__ void __launch_bounds__(GV_THREADS, sizeof(E) == 2 ? (TT == 1 ? 4 : 3) : 2)
-    gemv_dense_kernel(const GemvArgs a) {
+    gemv_dense_kernel(const GemvArgsOf<KIND> a) {
   extern __shared__ __align__(16) float xs[];
   __shared__ float red[GV_WARPS * GV_ROWS * TT > 32 ? GV_WARPS * GV_ROWS * TT : 32];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -229,7 +235,7 @@ __global__ void __launch_bounds__(GV_THREADS, sizeof(E) == 2 ? (TT == 1 ? 4 : 3)
   const E* w = static_cast<const E*>(a.w);
   float* out = a.out;
   int cta = blockIdx.x, ctas = gridDim.x;
-  if (KIND == GV_GROUPS_IN) {
+  if constexpr (KIND == GV_GROUPS_IN) {
     if (cta < a.store_ctas) {
       pdl_launch_dependents();
       const float2 turn = latent_turn(a.store, cta);
@@ -268,8 +274,11 @@ __global__ void __launch_bounds__(GV_THREADS, sizeof(E) == 2 ? (TT == 1 ? 4 : 3)
     finish_rows<GV_ROWS * TT>(acc, a.ks, red, [&](int grp, int idx, float v) {
       const int n = (base + grp) * GV_ROWS + idx / TT, t = idx % TT;
       if (n >= a.rows || t >= nt) return;
-      if (a.o.bias) v += a.o.bias[n];
-      out[(int64_t)(t0 + t) * a.out_ld + n] = a.o.relu2 ? relu_squared(v) : v;
+      if (KIND == GV_ROWS_IN) {
+        if (a.o.bias) v += a.o.bias[n];
+        if (a.o.relu2) v = relu_squared(v);
+      }
+      out[(int64_t)(t0 + t) * a.out_ld + n] = v;
     });
     if (nbase >= groups) break;
     base = nbase;
@@ -432,7 +441,7 @@ static unsigned gv_grid(const kanso_cuda_ctx* ctx, int64_t groups, int ks, int64
 }
 
 template <typename E, int TT, int KIND>
-static int32_t gemv_launch(kanso_cuda_ctx* ctx, const GemvArgs& a, dim3 grid, size_t smem) {
+static int32_t gemv_launch(kanso_cuda_ctx* ctx, const GemvArgsOf<KIND>& a, dim3 grid, size_t smem) {
   int32_t st = allow_max_smem(ctx, (const void*)gemv_dense_kernel<E, TT, KIND>);
   if (st) return st;
   const cudaError_t e =
@@ -441,10 +450,12 @@ static int32_t gemv_launch(kanso_cuda_ctx* ctx, const GemvArgs& a, dim3 grid, si
   return after_launch(ctx, "gemv_dense");
 }
 template <typename E, int TT>
-static int32_t gemv_launch(kanso_cuda_ctx* ctx, const GemvArgs& a, dim3 grid, size_t smem) {
+static int32_t gemv_launch(kanso_cuda_ctx* ctx, const GemvStoreArgs& a, dim3 grid, size_t smem) {
   if (a.s.gate) return gemv_launch<E, TT, GV_GATED_IN>(ctx, a, grid, smem);
   if (a.s.x_ld) return gemv_launch<E, TT, GV_GROUPS_IN>(ctx, a, grid, smem);
-  return gemv_launch<E, TT, GV_ROWS_IN>(ctx, a, grid, smem);
+  if (a.o.bias || a.o.relu2 || (a.s.y && a.s.form != Residual::kAdd))
+    return gemv_launch<E, TT, GV_ROWS_IN>(ctx, a, grid, smem);
+  return gemv_launch<E, TT, GV_PLAIN>(ctx, a, grid, smem);
 }
 
 int32_t launch_gemv(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat& w, const GemvSource& s,
@@ -456,10 +467,14 @@ int32_t launch_gemv(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat& w, con
     return fail(ctx, KANSO_ERR_UNSUPPORTED, "dense product: %lld columns", (long long)w.cols);
   const int64_t groups = (w.rows + GV_ROWS - 1) / GV_ROWS, copies = (T + tt - 1) / tt;
   const int64_t all = copies * w.groups;
-  if (w.groups > 65535 || ((w.groups > 1 || store) && (!s.x_ld || s.y)))
+  if (w.groups > 65535 || ((w.groups > 1 || store) && (!s.x_ld || s.y)) ||
+      ((s.x_ld || s.gate) && (o.bias || o.relu2)))
     return fail(ctx, KANSO_ERR_UNSUPPORTED, "dense product: %lld groups", (long long)w.groups);
-  GemvArgs a = {w.w, (int)w.rows, (int)w.cols, (int)w.ld, pick_ks(ctx, groups, all, w.ld / 8),
-                T, s, out, out_ld, o, store ? T : 0, store ? *store : LatentStore()};
+  GemvStoreArgs a;
+  static_cast<GemvArgs&>(a) = {w.w, (int)w.rows, (int)w.cols, (int)w.ld,
+                               pick_ks(ctx, groups, all, w.ld / 8), T, s, out, out_ld, o};
+  a.store_ctas = store ? T : 0;
+  if (store) a.store = *store;
   const dim3 grid(gv_grid(ctx, groups, a.ks, all) + a.store_ctas, (unsigned)copies,
                   (unsigned)w.groups);
   if (compute == KANSO_COMPUTE_BF16) {

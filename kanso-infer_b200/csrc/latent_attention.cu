@@ -65,8 +65,8 @@ __device__ __forceinline__ void latent_out(const LatentRowsArgs& p, int64_t i, i
     static_cast<E*>(p.r.out)[at] = to_elem<E>(v);
 }
 
-// The shares of one head of one row (blockIdx.x, blockIdx.y) in 128 of its columns (blockIdx.z): a
-// thread takes four of them from every eighth share.
+// The shares of one head of one row (blockIdx.x, blockIdx.y), 128 columns at a time (blockIdx.z and
+// on): a thread takes four of them from every eighth share.
 constexpr int LM_THREADS = 256, LM_COLS = 128, LM_GROUPS = LM_THREADS / (LM_COLS / 4);
 template <typename E>
 __global__ void __launch_bounds__(LM_THREADS) latent_merge_kernel(const LatentRowsArgs p) {
@@ -78,16 +78,18 @@ __global__ void __launch_bounds__(LM_THREADS) latent_merge_kernel(const LatentRo
   const uint32_t n = latent_span(p, i, 0).n_parts;
   const float* src = p.partial + ((size_t)i * p.a.heads + h) * p.parts * p.rec;
   float* dens = weight + p.parts;
-  const int q = tid % (LM_COLS / 4), g = tid / (LM_COLS / 4), c = blockIdx.z * LM_COLS + q * 4;
+  const int q = tid % (LM_COLS / 4), g = tid / (LM_COLS / 4);
   pdl_wait();
   float4 o[4];
-  // the first shares' sums are on their way while the weights are formed
+  auto first_shares = [&](int c) {
 #pragma unroll
-  for (int k = 0; k < 4; ++k) {
-    const uint32_t at = g + k * LM_GROUPS;
-    o[k] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (at < n && c < R) o[k] = *reinterpret_cast<const float4*>(src + (size_t)at * p.rec + c);
-  }
+    for (int k = 0; k < 4; ++k) {
+      const uint32_t at = g + k * LM_GROUPS;
+      o[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (at < n && c < R) o[k] = *reinterpret_cast<const float4*>(src + (size_t)at * p.rec + c);
+    }
+  };
+  first_shares(blockIdx.z * LM_COLS + q * 4);  // on their way while the weights are formed
   for (uint32_t k = tid; k < n; k += LM_THREADS) {
     const float2 m = *reinterpret_cast<const float2*>(src + (size_t)k * p.rec + p.rec - 4);
     weight[k] = m.x;
@@ -110,29 +112,34 @@ __global__ void __launch_bounds__(LM_THREADS) latent_merge_kernel(const LatentRo
     for (uint32_t k = tid; k < n; k += 32) weight[k] *= inv;
   }
   __syncthreads();
-  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-  for (uint32_t k0 = g; k0 < n; k0 += 4 * LM_GROUPS) {
+  for (int c0 = blockIdx.z * LM_COLS; c0 < R; c0 += gridDim.z * LM_COLS) {
+    const int c = c0 + q * 4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (uint32_t k0 = g; k0 < n; k0 += 4 * LM_GROUPS) {
 #pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      const uint32_t at = k0 + k * LM_GROUPS;
-      const float w = at < n ? weight[at] : 0.f;
-      if (at < n) {  // the pad behind the last column may hold anything
-        v.x = fmaf(w, o[k].x, v.x), v.y = fmaf(w, o[k].y, v.y);
-        v.z = fmaf(w, o[k].z, v.z), v.w = fmaf(w, o[k].w, v.w);
+      for (int k = 0; k < 4; ++k) {
+        const uint32_t at = k0 + k * LM_GROUPS;
+        if (at < n) {  // the pad behind the last column may hold anything
+          const float w = weight[at];
+          v.x = fmaf(w, o[k].x, v.x), v.y = fmaf(w, o[k].y, v.y);
+          v.z = fmaf(w, o[k].z, v.z), v.w = fmaf(w, o[k].w, v.w);
+        }
+        const uint32_t next = at + 4 * LM_GROUPS;
+        if (next < n && c < R)
+          o[k] = *reinterpret_cast<const float4*>(src + (size_t)next * p.rec + c);
       }
-      const uint32_t next = at + 4 * LM_GROUPS;
-      if (next < n && c < R)
-        o[k] = *reinterpret_cast<const float4*>(src + (size_t)next * p.rec + c);
     }
-  }
-  sums[g][q] = v;
-  __syncthreads();
-  const int col = blockIdx.z * LM_COLS + tid;
-  if (tid < LM_COLS && col < R) {
-    float t = 0.f;
+    first_shares(c + gridDim.z * LM_COLS);
+    sums[g][q] = v;
+    __syncthreads();
+    const int col = c0 + tid;
+    if (tid < LM_COLS && col < R) {
+      float t = 0.f;
 #pragma unroll
-    for (int k = 0; k < LM_GROUPS; ++k) t += reinterpret_cast<const float*>(sums[k])[tid];
-    latent_out<E>(p, i, h, col, t);
+      for (int k = 0; k < LM_GROUPS; ++k) t += reinterpret_cast<const float*>(sums[k])[tid];
+      latent_out<E>(p, i, h, col, t);
+    }
+    __syncthreads();
   }
 }
 
@@ -628,7 +635,9 @@ int32_t launch_latent_attn_rows(kanso_cuda_ctx* ctx, int32_t compute, const Late
   if (p.parts == 1) return KANSO_OK;
   auto merge =
       compute == KANSO_COMPUTE_BF16 ? latent_merge_kernel<bf16> : latent_merge_kernel<float>;
-  const dim3 mgrid(a.heads, (unsigned)r.n, (a.rank + LM_COLS - 1) / LM_COLS);
+  const uint32_t slabs = (a.rank + LM_COLS - 1) / LM_COLS;
+  const dim3 mgrid(a.heads, (unsigned)r.n,
+                   (uint64_t)a.heads * r.n * 2 > (uint64_t)ctx->sm_count * 8 ? 1 : slabs);
   const cudaError_t e =
       launch_dependent(ctx, merge, mgrid, dim3(LM_THREADS), (size_t)p.parts * 8, p);
   if (e != cudaSuccess) return cuda_fail(ctx, e, "latent merge launch");
