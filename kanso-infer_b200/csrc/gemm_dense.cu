@@ -454,8 +454,10 @@ int32_t launch_gemm(kanso_cuda_ctx* ctx, int32_t compute, const DenseMat& w, con
   if (!st) st = rows_map(ctx, x, r.T, w.cols, w.ld, nt, &xm);
   if (st) return st;
   const int64_t ty = tiles_of(r, nt), tx = (w.rows + 127) / 128;
-  const bool dual = nt == 128 && tx * ty >= 4 * (int64_t)ctx->sm_count;
   a.k_steps = (int)((w.cols + GD_K - 1) / GD_K);
+  // short products spend more time on their ends than the second tile saves: there two CTAs per
+  // SM, of which one stores while the other multiplies
+  const bool dual = nt == 128 && tx * ty >= 4 * (int64_t)ctx->sm_count && a.k_steps >= 12;
   // a share of the columns per CTA while the grid stays within one wave of two CTAs per SM
   int sp = 1;
   while (sp * 2 <= max_splits && tx * ty * sp * 2 <= 2 * (int64_t)ctx->sm_count &&
